@@ -2,7 +2,8 @@
 //   q heads: RMSNorm over the head (optional), rotation, written to q_out (which may be
 //            the projection itself: in place);
 //   k heads: RMSNorm (optional), rotation, written to the paged key cache;
-//   v heads: copied to the paged value cache.
+//   v heads: copied to the paged value cache, or first mixed with the same token's values of
+//            an earlier layer, v <- (1 - lambda) v + lambda v_first (struct VMix).
 // Restates infer/forward.odin:58-85 (norm before rotation, one [hd] weight shared
 // by all heads, half-split pairs (i, i + rot/2)) and the cache write of :47-49.
 // The rotation reads cos/sin of 32-bit angles from a table built on the host.
@@ -15,6 +16,15 @@
 
 #define HP_WARPS 4
 #define HP_MAX_HD 512
+
+// What happens to a value head on its way to the cache.  first: [rows][Hkv * vd] values of an earlier layer that are mixed
+// in (null: none); keep: where this layer's own values go for later layers, in the same layout (null: nowhere).
+template <typename T>
+struct VMix {
+    const T* first;
+    T* keep;
+    float lambda;
+};
 
 // TI: element type of the projection (bfloat16 or 32-bit; n_split 32-bit partial sums of a
 // split product are added first, in order).  T: element type of q_out and of the cache.
@@ -30,7 +40,7 @@ head_prep_kernel(const TI* qkv, int n_split, size_t split_stride, T* q_out,  // 
                  VecRef kw, int norm_mode, float eps, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                  int rot, int table_len, const int* __restrict__ tok_pos, const int* __restrict__ tok_seq,
                  const int* __restrict__ block_table, int bt_stride, T* __restrict__ k_cache,
-                 T* __restrict__ v_cache, int page_size, int write_kv, int pairs) {
+                 T* __restrict__ v_cache, int page_size, int write_kv, int pairs, VMix<T> vmix) {
     __shared__ float buf[HP_WARPS][HP_MAX_HD];
     __shared__ float whole_ss[2][HP_WARPS];
     pdl_trigger();
@@ -92,8 +102,14 @@ head_prep_kernel(const TI* qkv, int n_split, size_t split_stride, T* q_out,  // 
         b[j] = v;
         ss += v * v;
     }
-    if (is_v) {  // value head: stored as it is
-        for (int j = lane; j < n; j += 32) dst[j] = from_f32<T>(b[j]);
+    if (is_v) {  // value head: stored as it is, or mixed with an earlier layer's
+        const size_t at = ((size_t)t * Hkv + kvh) * vd;
+        for (int j = lane; j < n; j += 32) {
+            float v = b[j];
+            if (vmix.keep != nullptr) vmix.keep[at + j] = from_f32<T>(v);
+            if (vmix.first != nullptr) v = (1.0f - vmix.lambda) * v + vmix.lambda * to_f32(vmix.first[at + j]);
+            dst[j] = from_f32<T>(v);
+        }
         return;
     }
     if (norm_mode == 1) {
@@ -162,6 +178,19 @@ head_prep_kernel(const TI* qkv, int n_split, size_t split_stride, T* q_out,  // 
 using headmath::load_vec;
 using headmath::store_vec_bf16;
 
+// A value head's VEC elements of this lane on their way to the cache (see VMix); `at`: their place in its buffers.
+template <int VEC>
+__device__ __forceinline__ void value_to_cache(float (&v)[VEC], bf16* dst, const VMix<bf16>& vmix, size_t at) {
+    if (vmix.keep != nullptr) store_vec_bf16<VEC>(vmix.keep + at, v);
+    if (vmix.first != nullptr) {
+        float f[VEC];
+        load_vec<VEC>(vmix.first + at, f);
+#pragma unroll
+        for (int e = 0; e < VEC; ++e) v[e] = (1.0f - vmix.lambda) * v[e] + vmix.lambda * f[e];
+    }
+    store_vec_bf16<VEC>(dst, v);
+}
+
 // A warp per (token, head), TOK tokens per warp (one: for few tokens the kernel is a chain of
 // latencies, and everything that can be is fetched before the wait for the kernel before it).
 template <int VEC, typename TI, int TOK>
@@ -171,7 +200,7 @@ head_prep_fast_kernel(const TI* qkv, int n_split, size_t split_stride, bf16* q_o
                       const float* __restrict__ cos_t, const float* __restrict__ sin_t, int table_len,
                       const int* __restrict__ tok_pos, const int* __restrict__ tok_seq,
                       const int* __restrict__ block_table, int bt_stride, bf16* __restrict__ k_cache,
-                      bf16* __restrict__ v_cache, int page_size, int write_kv) {
+                      bf16* __restrict__ v_cache, int page_size, int write_kv, VMix<bf16> vmix) {
     constexpr int HD = VEC * 32, HALF = HD / 2;
     pdl_trigger();
     // What no earlier kernel of the step writes is fetched before the wait for that kernel: the
@@ -223,8 +252,8 @@ head_prep_fast_kernel(const TI* qkv, int n_split, size_t split_stride, bf16* q_o
 #pragma unroll
     for (int u = 0; u < TOK; ++u) {
         if (!active[u]) continue;
-        if (!is_q && !is_k) {  // value head: stored as it is
-            store_vec_bf16<VEC>(dst[u], v[u]);
+        if (!is_q && !is_k) {  // value head: no norm, no rotation
+            value_to_cache<VEC>(v[u], dst[u], vmix, ((size_t)(blockIdx.x * TOK + u) * Hkv + kvh) * HD + lane * VEC);
             continue;
         }
         float o[VEC];
@@ -243,7 +272,7 @@ head_prep_token_kernel(const TI* qkv, int n_split, size_t split_stride, bf16* q_
                        const float* __restrict__ cos_t, const float* __restrict__ sin_t, int table_len,
                        const int* __restrict__ tok_pos, const int* __restrict__ tok_seq,
                        const int* __restrict__ block_table, int bt_stride, bf16* __restrict__ k_cache,
-                       bf16* __restrict__ v_cache, int page_size, int write_kv) {
+                       bf16* __restrict__ v_cache, int page_size, int write_kv, VMix<bf16> vmix) {
     constexpr int HD = VEC * 32, HALF = HD / 2, UNROLL = 4;
     pdl_trigger();
     const int t = blockIdx.x;
@@ -298,8 +327,8 @@ head_prep_token_kernel(const TI* qkv, int n_split, size_t split_stride, bf16* q_
                 const int kvh = is_k ? head - Hq : head - Hq - Hkv;
                 dst = (is_k ? k_cache : v_cache) + (((size_t)page * Hkv + kvh) * page_size + (pos % page_size)) * HD + lane * VEC;
             }
-            if (!is_q && !is_k) {  // value head: stored as it is
-                store_vec_bf16<VEC>(dst, v[u]);
+            if (!is_q && !is_k) {  // value head: no norm, no rotation
+                value_to_cache<VEC>(v[u], dst, vmix, ((size_t)t * Hkv + (head - Hq - Hkv)) * HD + lane * VEC);
                 continue;
             }
             float o[VEC];
@@ -313,14 +342,15 @@ head_prep_token_kernel(const TI* qkv, int n_split, size_t split_stride, bf16* q_
 // elements apart).  q_out: [T, Hq hd] of dtype (row stride q_out_stride); it may be qkv
 // itself when there is one part of the same type (q is then normalised and rotated in place).
 // bias (null: none), norm_mode and vd as the general kernel describes them; the fast kernels take no
-// bias, norm_mode 0 or 1 and vd == hd.
+// bias, norm_mode 0 or 1 and vd == hd.  v_first, v_keep (each null: none; [T, Hkv vd] of dtype, contiguous), v_lambda: see VMix.
 extern "C" int odin_head_prep(const void* qkv, int in_dtype, int n_split, long long split_stride, void* q_out,
                               long long q_out_stride, int dtype, int T, int Hq, int Hkv, int hd, int vd,
                               long long row_stride, const void* bias, int bias_dtype, const void* q_norm_w,
                               const void* k_norm_w, int w_dtype, int norm_mode, float eps,
                               const float* cos_t, const float* sin_t, int rot, int table_len,
                               const int* tok_pos, const int* tok_seq, const int* block_table, int bt_stride,
-                              void* k_cache, void* v_cache, int page_size, int write_kv, int pairs, void* stream) {
+                              void* k_cache, void* v_cache, int page_size, int write_kv, int pairs, const void* v_first,
+                              void* v_keep, float v_lambda, void* stream) {
     if (T <= 0) return 0;
     if (hd > HP_MAX_HD || hd <= 0 || vd > HP_MAX_HD || vd <= 0 || (rot & 1) || rot > hd || rot < 0 || n_split < 1 ||
         norm_mode < 0 || norm_mode > 3)
@@ -336,19 +366,21 @@ extern "C" int odin_head_prep(const void* qkv, int in_dtype, int n_split, long l
     const bool fast_in = (in_dtype == ODIN_BF16 && n_split == 1) || in_dtype == ODIN_F32;
     if (plain_heads && fast_in && dtype == ODIN_BF16 && rot == hd && (hd == 64 || hd == 128) && (row_stride % 4) == 0 &&
         (split_stride % 4) == 0 && (q_out_stride % 4) == 0 &&
-        ((((uintptr_t)qkv) | ((uintptr_t)q_out) | ((uintptr_t)cos_t) | ((uintptr_t)sin_t)) & 15) == 0) {
+        ((((uintptr_t)qkv) | ((uintptr_t)q_out) | ((uintptr_t)cos_t) | ((uintptr_t)sin_t) | ((uintptr_t)v_first) |
+          ((uintptr_t)v_keep)) & 15) == 0) {
+        const VMix<bf16> vmix{(const bf16*)v_first, (bf16*)v_keep, v_lambda};
 #define FAST(VEC, TI, TOK)                                                                                         \
     odin_launch(head_prep_fast_kernel<VEC, TI, TOK>, dim3((T + TOK - 1) / TOK, grid.y), dim3(HP_WARPS * 32), 0, s,     \
                 (const TI*)qkv, n_split, (size_t)split_stride, (bf16*)q_out, (size_t)q_out_stride, T, Hq, Hkv,         \
                 (size_t)row_stride, qw, kw, has_norm, eps, cos_t, sin_t, table_len, tok_pos, tok_seq, block_table,      \
-                bt_stride, (bf16*)k_cache, (bf16*)v_cache, page_size, write_kv)
+                bt_stride, (bf16*)k_cache, (bf16*)v_cache, page_size, write_kv, vmix)
 #define FAST_T(VEC, TI)                                                                                            \
     do {                                                                                                           \
         if (T >= 256)                                                                                              \
             odin_launch(head_prep_token_kernel<VEC, TI>, dim3(T), dim3(HP_WARPS * 32), 0, s, (const TI*)qkv, n_split,  \
                         (size_t)split_stride, (bf16*)q_out, (size_t)q_out_stride, Hq, Hkv, (size_t)row_stride, qw, kw, \
                         has_norm, eps, cos_t, sin_t, table_len, tok_pos, tok_seq, block_table, bt_stride,              \
-                        (bf16*)k_cache, (bf16*)v_cache, page_size, write_kv);                                           \
+                        (bf16*)k_cache, (bf16*)v_cache, page_size, write_kv, vmix);                                     \
         else FAST(VEC, TI, 1);                                                                                     \
     } while (0)
         if (hd == 128 && in_dtype == ODIN_BF16) FAST_T(4, bf16);
@@ -364,7 +396,8 @@ extern "C" int odin_head_prep(const void* qkv, int in_dtype, int n_split, long l
     odin_launch(head_prep_kernel<TI, TT>, grid, dim3(HP_WARPS * 32), 0, s,                                           \
         (const TI*)qkv, n_split, (size_t)split_stride, (TT*)q_out, (size_t)q_out_stride, Hq, Hkv, hd, vd,           \
         (size_t)row_stride, bv, qw, kw, norm_mode, eps, cos_t, sin_t, rot, table_len, tok_pos, tok_seq, block_table,     \
-        (int)bt_stride, (TT*)k_cache, (TT*)v_cache, page_size, write_kv, pairs)
+        (int)bt_stride, (TT*)k_cache, (TT*)v_cache, page_size, write_kv, pairs,                                      \
+        VMix<TT>{(const TT*)v_first, (TT*)v_keep, v_lambda})
     if (in_dtype == ODIN_BF16 && dtype == ODIN_BF16) GO(bf16, bf16);
     else if (in_dtype == ODIN_F32 && dtype == ODIN_F32) GO(float, float);
     else if (in_dtype == ODIN_F32 && dtype == ODIN_BF16) GO(float, bf16);

@@ -6,7 +6,8 @@
 //                  [latent c (kv_rank) | rotated key part (rot)], which serves every head as key AND as value.
 //   heads_linear   a product per head: out[t, h, n] = sum_k a[t, h, k] * w[h][k][n].  With w = W_uk of head h it
 //                  turns a head's unrotated query into a query over the cached latent (q . (W_uk c) = (W_uk^T q) . c),
-//                  with w = W_uv^T of head h the attention's output over the latent into the head's value.
+//                  with w = W_uv^T of head h the attention's output over the latent into the head's value, times
+//                  sigmoid(gate[t, h]) where the heads are gated.
 //   rope_heads     rotation of the first `rot` elements of every head by the token's position, pairs (2i, 2i+1) or
 //                  (i, i + rot/2), the rest copied; an optional factor on the heads from a given one on.
 //
@@ -105,13 +106,37 @@ extern "C" int odin_latent_prep(const void* down, int in_dtype, int n_split, lon
 // ------------------------------------------------------------ a product per head
 // out[t, h, n] = sum_k a[t, h, k] * w[h][k][n]; a: row stride a_rs, head stride a_hs; out likewise; w: [H][K][N].
 // grid (N tiles of HL_THREADS, H, token tiles of HL_TOK); a thread owns one n for HL_TOK tokens and adds over k ascending.
+// a may be 32-bit partial sums of a split product (a_splits of them, a_ss elements apart, added in order); gate (optional):
+// a number per token and head, itself possibly partial sums; the sum is multiplied by its sigmoid.
 #define HL_THREADS 128
 #define HL_TOK 8
 
+struct HeadGate {
+    const void* p;             // null: no gate
+    int is_bf16, n_split;
+    long long split_stride, row_stride;
+    __device__ __forceinline__ float factor(int t, int h) const {
+        if (p == nullptr) return 1.0f;
+        float z = 0.f;
+        for (int s = 0; s < n_split; ++s) {
+            const size_t at = (size_t)s * split_stride + (size_t)t * row_stride + h;
+            z += is_bf16 ? __bfloat162float(((const bf16*)p)[at]) : ((const float*)p)[at];
+        }
+        return 1.0f / (1.0f + expf(-z));
+    }
+};
+
+template <typename TA>
+__device__ __forceinline__ float sum_parts(const TA* __restrict__ a, size_t at, int n_split, size_t split_stride) {
+    float v = to_f32(a[at]);
+    for (int s = 1; s < n_split; ++s) v += to_f32(a[(size_t)s * split_stride + at]);
+    return v;
+}
+
 template <typename TA, typename TW, typename TO>
 __global__ void __launch_bounds__(HL_THREADS)
-heads_linear_kernel(const TA* __restrict__ a, size_t a_rs, size_t a_hs, const TW* __restrict__ w, TO* __restrict__ out,
-                    size_t o_rs, size_t o_hs, int T, int N, int K) {
+heads_linear_kernel(const TA* __restrict__ a, int a_splits, size_t a_ss, size_t a_rs, size_t a_hs, const TW* __restrict__ w,
+                    TO* __restrict__ out, size_t o_rs, size_t o_hs, int T, int N, int K, HeadGate gate) {
     extern __shared__ __align__(16) float as[];   // [K][HL_TOK]
     pdl_trigger();
     const int h = blockIdx.y, t0 = blockIdx.z * HL_TOK;
@@ -119,7 +144,7 @@ heads_linear_kernel(const TA* __restrict__ a, size_t a_rs, size_t a_hs, const TW
     pdl_wait();
     for (int e = threadIdx.x; e < K * HL_TOK; e += blockDim.x) {
         const int u = e / K, k = e % K;
-        as[k * HL_TOK + u] = (t0 + u < T) ? to_f32(a[(size_t)(t0 + u) * a_rs + (size_t)h * a_hs + k]) : 0.f;
+        as[k * HL_TOK + u] = (t0 + u < T) ? sum_parts(a, (size_t)(t0 + u) * a_rs + (size_t)h * a_hs + k, a_splits, a_ss) : 0.f;
     }
     __syncthreads();
     if (n >= N) return;
@@ -149,7 +174,7 @@ heads_linear_kernel(const TA* __restrict__ a, size_t a_rs, size_t a_hs, const TW
     }
 #pragma unroll
     for (int u = 0; u < HL_TOK; ++u)
-        if (t0 + u < T) out[(size_t)(t0 + u) * o_rs + (size_t)h * o_hs + n] = from_f32<TO>(acc[u]);
+        if (t0 + u < T) out[(size_t)(t0 + u) * o_rs + (size_t)h * o_hs + n] = from_f32<TO>(acc[u] * gate.factor(t0 + u, h));
 }
 
 // Many tokens: a CTA takes 64 tokens by 64 output channels of one head, K in steps of 32 through shared memory, a thread
@@ -159,8 +184,9 @@ heads_linear_kernel(const TA* __restrict__ a, size_t a_rs, size_t a_hs, const TW
 #define HLT_KC 32
 template <typename TA, typename TW, typename TO>
 __global__ void __launch_bounds__(256)
-heads_linear_tiled_kernel(const TA* __restrict__ a, size_t a_rs, size_t a_hs, const TW* __restrict__ w, TO* __restrict__ out,
-                          size_t o_rs, size_t o_hs, int T, int N, int K) {
+heads_linear_tiled_kernel(const TA* __restrict__ a, int a_splits, size_t a_ss, size_t a_rs, size_t a_hs,
+                          const TW* __restrict__ w, TO* __restrict__ out, size_t o_rs, size_t o_hs, int T, int N, int K,
+                          HeadGate gate) {
     __shared__ __align__(16) float As[HLT_KC][HLT_TILE + 4];   // [k][token]
     __shared__ __align__(16) float Ws[HLT_KC][HLT_TILE];       // [k][channel]
     pdl_trigger();
@@ -179,7 +205,7 @@ heads_linear_tiled_kernel(const TA* __restrict__ a, size_t a_rs, size_t a_hs, co
         for (int f = 0; f < 8; ++f) {
             const int e = threadIdx.x + f * 256;
             const int u = e / HLT_KC, k = e % HLT_KC;          // a: consecutive threads along k
-            ra[f] = (t0 + u < T && k0 + k < K) ? to_f32(a[(size_t)(t0 + u) * a_rs + (size_t)h * a_hs + k0 + k]) : 0.f;
+            ra[f] = (t0 + u < T && k0 + k < K) ? sum_parts(a, (size_t)(t0 + u) * a_rs + (size_t)h * a_hs + k0 + k, a_splits, a_ss) : 0.f;
             const int kw = e / HLT_TILE, n = e % HLT_TILE;     // w: consecutive threads along the channels
             rw[f] = (k0 + kw < K && n0 + n < N) ? to_f32(wh[(size_t)(k0 + kw) * N + n0 + n]) : 0.f;
         }
@@ -206,18 +232,22 @@ heads_linear_tiled_kernel(const TA* __restrict__ a, size_t a_rs, size_t a_hs, co
     for (int i = 0; i < 4; ++i) {
         const int t = t0 + ty * 4 + i;
         if (t >= T) continue;
+        const float f = gate.factor(t, h);
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx * 4 + j;
-            if (n < N) out[(size_t)t * o_rs + (size_t)h * o_hs + n] = from_f32<TO>(acc[i][j]);
+            if (n < N) out[(size_t)t * o_rs + (size_t)h * o_hs + n] = from_f32<TO>(acc[i][j] * f);
         }
     }
 }
 
-extern "C" int odin_heads_linear(const void* a, int a_dtype, long long a_rs, long long a_hs, const void* w, int w_dtype,
-                                 void* out, int out_dtype, long long o_rs, long long o_hs, int T, int H, int N, int K,
-                                 void* stream) {
+extern "C" int odin_heads_linear(const void* a, int a_dtype, int a_splits, long long a_ss, long long a_rs, long long a_hs,
+                                 const void* w, int w_dtype, void* out, int out_dtype, long long o_rs, long long o_hs, int T,
+                                 int H, int N, int K, const void* gate, int gate_dtype, int gate_splits, long long gate_ss,
+                                 long long gate_rs, void* stream) {
     if (T <= 0) return 0;
+    if (a_splits < 1 || (gate != nullptr && gate_splits < 1)) return ODIN_ERR_BAD_ARG;
+    const HeadGate hg{gate, gate_dtype == ODIN_BF16, gate_splits, gate_ss, gate_rs};
     if (H <= 0 || H > 65535 || N <= 0 || K <= 0) return ODIN_ERR_BAD_ARG;
     const size_t smem = (size_t)K * HL_TOK * sizeof(float);
     if (smem > 48 * 1024 || (T + HL_TOK - 1) / HL_TOK > 65535) return ODIN_ERR_UNSUPPORTED;
@@ -228,11 +258,13 @@ extern "C" int odin_heads_linear(const void* a, int a_dtype, long long a_rs, lon
 #define GO(TA, TW, TO)                                                                                              \
     do {                                                                                                            \
         if (tiled)                                                                                                  \
-            odin_launch(heads_linear_tiled_kernel<TA, TW, TO>, tgrid, dim3(256), 0, s, (const TA*)a, (size_t)a_rs,  \
-                        (size_t)a_hs, (const TW*)w, (TO*)out, (size_t)o_rs, (size_t)o_hs, T, N, K);                 \
+            odin_launch(heads_linear_tiled_kernel<TA, TW, TO>, tgrid, dim3(256), 0, s, (const TA*)a, a_splits,      \
+                        (size_t)a_ss, (size_t)a_rs, (size_t)a_hs, (const TW*)w, (TO*)out, (size_t)o_rs,             \
+                        (size_t)o_hs, T, N, K, hg);                                                                 \
         else                                                                                                        \
-            odin_launch(heads_linear_kernel<TA, TW, TO>, grid, dim3(HL_THREADS), smem, s, (const TA*)a,             \
-                        (size_t)a_rs, (size_t)a_hs, (const TW*)w, (TO*)out, (size_t)o_rs, (size_t)o_hs, T, N, K);   \
+            odin_launch(heads_linear_kernel<TA, TW, TO>, grid, dim3(HL_THREADS), smem, s, (const TA*)a, a_splits,   \
+                        (size_t)a_ss, (size_t)a_rs, (size_t)a_hs, (const TW*)w, (TO*)out, (size_t)o_rs,             \
+                        (size_t)o_hs, T, N, K, hg);                                                                 \
     } while (0)
     if (a_dtype == ODIN_BF16 && w_dtype == ODIN_BF16 && out_dtype == ODIN_BF16) GO(bf16, bf16, bf16);
     else if (a_dtype == ODIN_F32 && w_dtype == ODIN_F32 && out_dtype == ODIN_F32) GO(float, float, float);

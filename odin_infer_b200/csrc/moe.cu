@@ -12,8 +12,9 @@
 //             bias), a group's score is its largest choice score, and the weights are the chosen experts' scores (without the
 //             correction) divided by their sum (+ 1e-20), times `route_scale`.  Rows from `n_real` on have no expert behind
 //             them: a token that chooses one gets its own input back, times the weight (summed per token into `pass_out`).
+//             score 3: the scores are sigmoid(z); the weights are the chosen experts' scores themselves, times `route_scale`.
 //   gate|up:  a[r, j] = act(Wg[e_r] h_t)_j * (Wu[e_r] h_t)_j          r = t * rows_per_token + k
-//             (not gated: a[r, j] = act(Wu[e_r] h_t)_j)
+//             (not gated: a[r, j] = act(Wu[e_r] h_t)_j; with weights on the input h_t is weight_r h_t, and `down` weighs nothing)
 //   down:     y[k, t, :] = weight_r * Wd[e_r] a[r, :]                 32-bit, one slice per choice
 //
 // The slices y[k] are partial sums of the layer's update: whoever adds the update adds them in the
@@ -227,7 +228,8 @@ moe_router_kernel(const TH* __restrict__ h, size_t h_stride, const TW* __restric
                 if (ov > best || (ov == best && oe < best_e)) { best = ov; best_e = oe; }
             }
             if (k == 0) first = best;
-            const float p = score == 1 ? best : score == 2 ? (best_e < E ? sc[best_e] : 0.f) : expf(best - first);
+            const float p = score == 1 ? best : score == 2 ? (best_e < E ? sc[best_e] : 0.f)
+                          : score == 3 ? 1.0f / (1.0f + expf(-best)) : expf(best - first);
             sum += p;
             if (lane == k) { chosen = p; chosen_id = best_e; }
             if (lane == 0 && best_e < E) z[best_e] = -CUDART_INF_F;
@@ -235,7 +237,7 @@ moe_router_kernel(const TH* __restrict__ h, size_t h_stride, const TW* __restric
         }
         // rows from n_real on have no expert behind them: their weights are summed into pass_out (the token's input is
         // handed through that many times) and their places name no expert
-        const float wt = score != 0 ? chosen / (sum + 1e-20f) * route_scale : chosen / sum;
+        const float wt = score == 3 ? chosen * route_scale : score != 0 ? chosen / (sum + 1e-20f) * route_scale : chosen / sum;
         const bool passes = lane < top && chosen_id >= n_real && chosen_id < E;
         const float passed = warp_sum(passes ? wt : 0.f);
         if (pass_out != nullptr && lane == 0) pass_out[t] = passed;
@@ -256,7 +258,7 @@ extern "C" int odin_moe_router(const void* h, int h_dtype, long long h_stride, c
                                int gate_row, float* gate_out, int n_real, float* pass_out, void* stream) {
     if (T <= 0) return 0;
     if (E <= 0 || top <= 0 || top > 32 || top > E || always < 0 || d <= 0) return ODIN_ERR_UNSUPPORTED;
-    if (score < 0 || score > 2 || n_real < 0 || n_real > E || (n_real < E && pass_out == nullptr)) return ODIN_ERR_BAD_ARG;
+    if (score < 0 || score > 3 || n_real < 0 || n_real > E || (n_real < E && pass_out == nullptr)) return ODIN_ERR_BAD_ARG;
     if (groups < 1 || groups > 32 || E % groups != 0 || keep < 1 || keep > groups || (long long)keep * (E / groups) < top)
         return ODIN_ERR_UNSUPPORTED;
     const size_t smem = (size_t)(d + 2 * E + 1) * sizeof(float);
@@ -289,8 +291,8 @@ extern "C" int odin_moe_router(const void* h, int h_dtype, long long h_stride, c
 // grid (rows, column blocks).  w: [experts][2 ff][d], the ff gate rows before the ff up rows (not gated: [experts][ff][d]).
 template <typename TH, typename TW>
 __global__ void __launch_bounds__(MOE_THREADS)
-moe_gate_up_kernel(const TH* __restrict__ h, size_t h_stride, const TW* __restrict__ w, const int* __restrict__ ids, int per,
-                   int ff, int d, int act, int gated, TH* __restrict__ out) {
+moe_gate_up_kernel(const TH* __restrict__ h, size_t h_stride, const TW* __restrict__ w, const int* __restrict__ ids,
+                   const float* __restrict__ in_wts, int per, int ff, int d, int act, int gated, TH* __restrict__ out) {
     extern __shared__ float hrow[];  // d
     pdl_trigger();
     pdl_wait();
@@ -303,7 +305,8 @@ moe_gate_up_kernel(const TH* __restrict__ h, size_t h_stride, const TW* __restri
         for (int j = c0 + threadIdx.x; j < min(ff, c0 + MOE_COLS); j += blockDim.x) orow[j] = from_f32<TH>(0.f);
         return;
     }
-    for (int i = threadIdx.x; i < d; i += blockDim.x) hrow[i] = to_f32(h[(size_t)t * h_stride + i]);
+    const float wt = in_wts != nullptr ? in_wts[r] : 1.0f;
+    for (int i = threadIdx.x; i < d; i += blockDim.x) hrow[i] = wt * to_f32(h[(size_t)t * h_stride + i]);
     __syncthreads();
     const TW* we = w + (size_t)e * (gated ? 2 : 1) * ff * d;
     for (int j = c0 + warp; j < min(ff, c0 + MOE_COLS); j += MOE_WARPS) {
@@ -314,7 +317,7 @@ moe_gate_up_kernel(const TH* __restrict__ h, size_t h_stride, const TW* __restri
 }
 
 extern "C" int odin_moe_gate_up(const void* h, int h_dtype, long long h_stride, const void* w, int w_dtype, const int* ids,
-                                int T, int per, int ff, int d, int act, int gated, void* out, void* stream) {
+                                const float* in_wts, int T, int per, int ff, int d, int act, int gated, void* out, void* stream) {
     if (T <= 0 || per <= 0) return 0;
     if (act != MOE_ACT_SILU && act != MOE_ACT_GELU_TANH && act != MOE_ACT_RELU2) return ODIN_ERR_BAD_ARG;
     const size_t smem = (size_t)d * sizeof(float);
@@ -326,7 +329,7 @@ extern "C" int odin_moe_gate_up(const void* h, int h_dtype, long long h_stride, 
         if (smem > 48 * 1024)                                                                                         \
             cudaFuncSetAttribute(moe_gate_up_kernel<TH, TW>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
         odin_launch(moe_gate_up_kernel<TH, TW>, grid, dim3(MOE_THREADS), smem, s, (const TH*)h, (size_t)h_stride,     \
-                    (const TW*)w, ids, per, ff, d, act, gated, (TH*)out);                                             \
+                    (const TW*)w, ids, in_wts, per, ff, d, act, gated, (TH*)out);                                     \
     } while (0)
     if (h_dtype == ODIN_BF16 && w_dtype == ODIN_BF16) GO(bf16, bf16);
     else if (h_dtype == ODIN_F32 && w_dtype == ODIN_F32) GO(float, float);
@@ -358,7 +361,7 @@ moe_down_kernel(const TA* __restrict__ a, const TW* __restrict__ w, const int* _
     }
     for (int i = threadIdx.x; i < ff; i += blockDim.x) arow[i] = to_f32(a[(size_t)r * ff + i]);
     __syncthreads();
-    const float wt = wts[r];
+    const float wt = wts != nullptr ? wts[r] : 1.0f;
     const TW* we = w + (size_t)e * d * ff;
     for (int c = c0 + warp; c < min(d, c0 + MOE_COLS); c += MOE_WARPS) {
         const float s = warp_dot(we + (size_t)c * ff, arow, ff, lane);

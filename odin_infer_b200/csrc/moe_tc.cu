@@ -99,22 +99,37 @@ moe_plan_kernel(const int* __restrict__ ids, int rows, int n_experts, int* __res
 }
 
 // ------------------------------------------------------------------------------------------------ gather
-// A block takes GATHER_PLACES places; their row numbers, then their rows' loads go out together.
+// A block takes GATHER_PLACES places; their row numbers, then their rows' loads go out together.  in_wts (optional): a
+// row (token, choice) is multiplied by its weight on the way (a 32-bit product, rounded once).
 constexpr int GATHER_PLACES = 4;
 __global__ void __launch_bounds__(256)
 moe_gather_kernel(const bf16* __restrict__ h, size_t h_stride, const int* __restrict__ row_of_place, int places, int per, int d,
-                  bf16* __restrict__ out) {
+                  const float* __restrict__ in_wts, bf16* __restrict__ out) {
     pdl_trigger();
     pdl_wait();
     const int p0 = blockIdx.x * GATHER_PLACES;
     int r[GATHER_PLACES];
 #pragma unroll
     for (int k = 0; k < GATHER_PLACES; ++k) r[k] = (p0 + k < places) ? row_of_place[p0 + k] : -2;
+    float wt[GATHER_PLACES];
+#pragma unroll
+    for (int k = 0; k < GATHER_PLACES; ++k) wt[k] = (in_wts != nullptr && r[k] >= 0) ? in_wts[r[k]] : 1.0f;
     for (int i = threadIdx.x * 8; i < d; i += blockDim.x * 8) {
         uint4 v[GATHER_PLACES];
 #pragma unroll
         for (int k = 0; k < GATHER_PLACES; ++k)
             v[k] = r[k] >= 0 ? *reinterpret_cast<const uint4*>(h + (size_t)(r[k] / per) * h_stride + i) : make_uint4(0, 0, 0, 0);
+        if (in_wts != nullptr) {
+#pragma unroll
+            for (int k = 0; k < GATHER_PLACES; ++k) {
+                __nv_bfloat162* q = reinterpret_cast<__nv_bfloat162*>(&v[k]);
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const float2 f = __bfloat1622float2(q[j]);
+                    q[j] = __floats2bfloat162_rn(wt[k] * f.x, wt[k] * f.y);
+                }
+            }
+        }
 #pragma unroll
         for (int k = 0; k < GATHER_PLACES; ++k)
             if (r[k] != -2) *reinterpret_cast<uint4*>(out + (size_t)(p0 + k) * d + i) = v[k];
@@ -133,7 +148,7 @@ moe_combine_kernel(const float* __restrict__ c, const int* __restrict__ place_of
         for (int k = 0; k < per; ++k) {
             const int place = place_of_row[t * per + k];
             if (place < 0) continue;
-            const float w = wts[t * per + k];
+            const float w = wts != nullptr ? wts[t * per + k] : 1.0f;
             const float4 v = *reinterpret_cast<const float4*>(c + (size_t)place * d + i);
             acc.x = fmaf(w, v.x, acc.x); acc.y = fmaf(w, v.y, acc.y); acc.z = fmaf(w, v.z, acc.z); acc.w = fmaf(w, v.w, acc.w);
         }
@@ -419,12 +434,12 @@ extern "C" int odin_moe_plan(const int* ids, int rows, int n_experts, int* place
     return 0;
 }
 
-extern "C" int odin_moe_gather(const void* h, long long h_stride, const int* row_of_place, int places, int per, int d, void* out,
-                               void* stream) {
+extern "C" int odin_moe_gather(const void* h, long long h_stride, const int* row_of_place, int places, int per, int d,
+                               const float* in_wts, void* out, void* stream) {
     if (places <= 0) return 0;
     if (d % 8 != 0 || h_stride % 8 != 0 || ((((uintptr_t)h) | ((uintptr_t)out)) & 15) != 0) return ODIN_ERR_UNSUPPORTED;
     odin_launch(moe_gather_kernel, dim3((places + GATHER_PLACES - 1) / GATHER_PLACES), dim3(256), 0, (cudaStream_t)stream,
-                (const bf16*)h, (size_t)h_stride, row_of_place, places, per, d, (bf16*)out);
+                (const bf16*)h, (size_t)h_stride, row_of_place, places, per, d, in_wts, (bf16*)out);
     ODIN_LAUNCH_CHECK();
     return 0;
 }

@@ -301,6 +301,11 @@ def softcap(z: torch.Tensor, cap: float, scale: float = 1.0) -> None:
                                           c_float(cap), c_float(scale), _stream()), "softcap")
 
 
+def _vec(w: torch.Tensor | None) -> tuple:
+    """A weight vector's pointer and element type (null where there is none)."""
+    return _ptr(w), c_int(dtype_code(w.dtype) if w is not None else 0)
+
+
 class Term:
     """One term of a combined update (see `combine_add`): `value` [n, d] or [parts, n, d] partial sums, times `scale`,
     times row_scale[r] (float32 [n]) where given; with norm_weight ([d]) the summed row is first divided by its root mean
@@ -314,11 +319,14 @@ class Term:
 
 def combine_add(x: torch.Tensor | None, terms: list, post_weight: torch.Tensor | None = None, post_eps: float = 0.0,
                 next_weight: torch.Tensor | None = None, next_eps: float = 0.0, out: torch.Tensor | None = None,
-                rows: torch.Tensor | None = None, tok_seq: torch.Tensor | None = None) -> None:
+                rows: torch.Tensor | None = None, tok_seq: torch.Tensor | None = None, post_bias: torch.Tensor | None = None,
+                post_center: bool = False, next_bias: torch.Tensor | None = None, next_center: bool = False) -> None:
     """y = the sum of up to four `Term`s; x += post_weight * y / rms(y) (post_weight None: x += y), in place unless `rows`
-    gathers; then out = next_weight * x / rms(x) where next_weight is given.  x None: out (float32) = y.  Rows of sequence
+    gathers; then, where `out` is given, out = next_weight * x / rms(x), or x converted where next_weight is None.
+    post_center / next_center: the norm is a layer norm (the row's mean is taken off first, the variance is the mean of the
+    squared deviations); post_bias / next_bias: added after the weight.  x None: out (float32) = y.  Rows of sequence
     -1 (tok_seq) are skipped.  All sums 32-bit, in an order that the width fixes."""
-    assert 0 < len(terms) <= 4
+    assert len(terms) <= 4
     ref = x if x is not None else out
     d = ref.shape[-1]
     n_all = x.shape[0] if x is not None else out.shape[0]
@@ -343,12 +351,13 @@ def combine_add(x: torch.Tensor | None, terms: list, post_weight: torch.Tensor |
             assert t.norm_weight.numel() == d and t.norm_weight.is_contiguous()
         nws[i], nwd[i] = _ptr(t.norm_weight), dtype_code(t.norm_weight.dtype) if t.norm_weight is not None else 0
         nep[i] = t.norm_eps
-    for w in (post_weight, next_weight):
+    for w in (post_weight, next_weight, post_bias, next_bias):
         assert w is None or (w.numel() == d and w.is_contiguous())
+    assert (post_bias is None or post_weight is not None) and (next_bias is None or next_weight is not None)
     _check(_fn("rowwise", "odin_combine_add")(
-        _ptr(x), c_int(n), ptrs, dts, nsp, sst, scl, rsc, nws, nwd, nep, _ptr(post_weight),
-        c_int(dtype_code(post_weight.dtype) if post_weight is not None else 0), c_float(post_eps), _ptr(next_weight),
-        c_int(dtype_code(next_weight.dtype) if next_weight is not None else 0), c_float(next_eps), _ptr(out),
+        _ptr(x), c_int(n), ptrs, dts, nsp, sst, scl, rsc, nws, nwd, nep, *_vec(post_weight), *_vec(post_bias),
+        c_float(post_eps), c_int(1 if post_center else 0), *_vec(next_weight), *_vec(next_bias), c_float(next_eps),
+        c_int(1 if next_center else 0), _ptr(out),
         c_int(dtype_code(out.dtype) if out is not None else 0), _ptr(rows), _ptr(tok_seq), c_int(n_rows), c_int(d),
         _stream()), "combine_add")
 
@@ -370,6 +379,7 @@ def moe_router(h: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None, top:
     1e-20) * route_scale.  n_real: the first n_real rows of W have experts behind them; a token that chooses a later row
     gets its own input back times that weight: such places name expert -1 with weight 0, and the token's summed weight of
     them goes to pass_out (float32 [T]).  The `always` choices name the experts n_real, n_real + 1, ...
+    score "sigmoid_as_is": the `top` largest sigmoid(z + bias) are chosen, and their weights are these scores * route_scale.
     gate_row: W has one row more than there are experts, g; the `always` choices are weighted by sigmoid(g . h),
     which also goes to gate_out (float32 [T]) where given."""
     T, d = h.shape
@@ -394,31 +404,38 @@ def moe_router(h: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None, top:
         "moe_router")
 
 
-ROUTER_SCORES = {"softmax_of_chosen": 0, "sigmoid_in_groups": 1, "softmax_corrected_in_groups": 2}
+ROUTER_SCORES = {"softmax_of_chosen": 0, "sigmoid_in_groups": 1, "softmax_corrected_in_groups": 2, "sigmoid_as_is": 3}
 
 
-def moe_gate_up(h: torch.Tensor, w: torch.Tensor, ids: torch.Tensor, kind: str, out: torch.Tensor, gated: bool = True) -> None:
+def _wts(wts: torch.Tensor | None, ids: torch.Tensor) -> c_void_p:
+    assert wts is None or (wts.dtype == torch.float32 and wts.is_contiguous() and wts.shape == ids.shape)
+    return _ptr(wts)
+
+
+def moe_gate_up(h: torch.Tensor, w: torch.Tensor, ids: torch.Tensor, kind: str, out: torch.Tensor, gated: bool = True,
+                in_wts: torch.Tensor | None = None) -> None:
     """out[t * per + k, :] = act(Wg[e] h[t]) * (Wu[e] h[t]) with e = ids[t, k]; w: [experts, 2 ff, d], gate rows first.
-    Not gated: out[t * per + k, :] = act(W[e] h[t]), w: [experts, ff, d]."""
+    Not gated: out[t * per + k, :] = act(W[e] h[t]), w: [experts, ff, d].  in_wts (float32 [T, per]): the expert reads
+    in_wts[t, k] * h[t]."""
     T, d = h.shape
     per, ff = ids.shape[1], out.shape[1]
     assert h.stride(1) == 1 and w.is_contiguous() and tuple(w.shape[1:]) == ((2 if gated else 1) * ff, d) and out.is_contiguous()
     assert out.shape[0] == T * per and out.dtype == h.dtype and ids.dtype == torch.int32 and ids.is_contiguous()
     _check(_fn("moe", "odin_moe_gate_up")(
         _ptr(h), c_int(dtype_code(h.dtype)), c_longlong(h.stride(0)), _ptr(w), c_int(dtype_code(w.dtype)), _ptr(ids),
-        c_int(T), c_int(per), c_int(ff), c_int(d), c_int(ACTIVATIONS[kind]), c_int(1 if gated else 0), _ptr(out),
+        _wts(in_wts, ids), c_int(T), c_int(per), c_int(ff), c_int(d), c_int(ACTIVATIONS[kind]), c_int(1 if gated else 0), _ptr(out),
         _stream()), "moe_gate_up")
 
 
-def moe_down(a: torch.Tensor, w: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor, out: torch.Tensor) -> None:
+def moe_down(a: torch.Tensor, w: torch.Tensor, ids: torch.Tensor, wts: torch.Tensor | None, out: torch.Tensor) -> None:
     """out[k, t, :] = wts[t, k] * Wd[e] a[t * per + k] with e = ids[t, k]; w: [experts, d, ff]; out float32 [per, T, d]:
-    partial sums of the tokens' update."""
+    partial sums of the tokens' update.  wts None: weights of one."""
     T, per = ids.shape
     ff, d = a.shape[1], w.shape[1]
     assert a.is_contiguous() and a.shape[0] == T * per and w.is_contiguous() and w.shape[2] == ff
     assert out.dtype == torch.float32 and out.is_contiguous() and tuple(out.shape) == (per, T, d)
     _check(_fn("moe", "odin_moe_down")(
-        _ptr(a), c_int(dtype_code(a.dtype)), _ptr(w), c_int(dtype_code(w.dtype)), _ptr(ids), _ptr(wts), c_int(T),
+        _ptr(a), c_int(dtype_code(a.dtype)), _ptr(w), c_int(dtype_code(w.dtype)), _ptr(ids), _wts(wts, ids), c_int(T),
         c_int(per), c_int(ff), c_int(d), _ptr(out), _stream()), "moe_down")
 
 
@@ -447,11 +464,14 @@ def moe_plan(ids: torch.Tensor, n_experts: int, place_of_row: torch.Tensor, row_
                                           c_int(row_of_place.numel()), _ptr(tile_expert), _stream()), "moe_plan")
 
 
-def moe_gather(h: torch.Tensor, row_of_place: torch.Tensor, per: int, out: torch.Tensor) -> None:
-    """out[place] = h[row_of_place[place] // per] (bfloat16), zeros where the place is padding."""
+def moe_gather(h: torch.Tensor, row_of_place: torch.Tensor, per: int, out: torch.Tensor,
+               in_wts: torch.Tensor | None = None) -> None:
+    """out[place] = h[row_of_place[place] // per] (bfloat16), zeros where the place is padding.  in_wts (float32, one per
+    row): row r is multiplied by in_wts[r], in 32-bit, and rounded once."""
     assert h.dtype == out.dtype == torch.bfloat16 and out.is_contiguous() and out.shape == (row_of_place.numel(), h.shape[1])
+    assert in_wts is None or (in_wts.dtype == torch.float32 and in_wts.is_contiguous())
     _check(_fn("moe_tc", "odin_moe_gather")(_ptr(h), c_longlong(h.stride(0)), _ptr(row_of_place), c_int(out.shape[0]),
-                                            c_int(per), c_int(h.shape[1]), _ptr(out), _stream()), "moe_gather")
+                                            c_int(per), c_int(h.shape[1]), _ptr(in_wts), _ptr(out), _stream()), "moe_gather")
 
 
 def moe_grouped(a: torch.Tensor, w: torch.Tensor, tile_expert: torch.Tensor, out: torch.Tensor, kind: str | None = None,
@@ -482,12 +502,14 @@ def moe_grouped(a: torch.Tensor, w: torch.Tensor, tile_expert: torch.Tensor, out
         c_longlong(out.stride(0)), _stream()), "moe_grouped")
 
 
-def moe_combine(c: torch.Tensor, place_of_row: torch.Tensor, wts: torch.Tensor, out: torch.Tensor) -> None:
-    """out[t] = sum_k wts[t, k] * c[place_of_row[t * per + k]] (float32), the choices in their order."""
-    T, per = wts.shape
-    d = c.shape[1]
-    assert c.dtype == out.dtype == wts.dtype == torch.float32 and c.is_contiguous() and out.is_contiguous()
-    assert tuple(out.shape) == (T, d) and place_of_row.numel() == T * per and wts.is_contiguous()
+def moe_combine(c: torch.Tensor, place_of_row: torch.Tensor, wts: torch.Tensor | None, out: torch.Tensor) -> None:
+    """out[t] = sum_k wts[t, k] * c[place_of_row[t * per + k]] (float32), the choices in their order (wts None: weights
+    of one)."""
+    T, d = out.shape
+    per = place_of_row.numel() // T
+    assert c.dtype == out.dtype == torch.float32 and c.is_contiguous() and out.is_contiguous() and c.shape[1] == d
+    assert place_of_row.numel() == T * per
+    assert wts is None or (wts.dtype == torch.float32 and tuple(wts.shape) == (T, per) and wts.is_contiguous())
     _check(_fn("moe_tc", "odin_moe_combine")(_ptr(c), _ptr(place_of_row), _ptr(wts), c_int(T), c_int(per), c_int(d),
                                              _ptr(out), _stream()), "moe_combine")
 
@@ -582,6 +604,46 @@ def linear_recurrence(mode: str, q: torch.Tensor, k: torch.Tensor | None, g: tor
         c_longlong(shift_state.stride(0) if shift_state is not None else 0), c_int(width), c_int(block_len),
         c_int(n_blocks), _ptr(qp), _ptr(s_loc), _ptr(d_tot), c_float(q_scale), c_int(heads_per_group), _stream()),
         "linear_recurrence", kernels=kernels)
+
+
+def delta_rule(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a: torch.Tensor, b: torch.Tensor, A_log: torch.Tensor,
+               a_bias: torch.Tensor, out: torch.Tensor, state: torch.Tensor, seq_start: torch.Tensor,
+               seq_slots: torch.Tensor, n_seqs: int, n_heads: int, dk: int, dv: int, heads_per_group: int = 1,
+               q_scale: float = 1.0, unit_eps: float = 1e-6, block_len: int = 0, max_new: int = 0) -> None:
+    """The gated delta rule over a state S [dk, dv] per (sequence, head) in `state` (float32 [slots, >= H dk dv], any row
+    stride), sequence t's rows in order.  With u(x) = x / sqrt(sum(x^2) + unit_eps) over a head's dk elements,
+    g = exp(-exp(A_log[h]) softplus(a[t, h] + a_bias[h])) and beta = sigmoid(b[t, h]):
+
+        S <- g S;   w = beta (v - S^T u(k));   S <- S + u(k) w^T;   o = S^T (q_scale u(q))
+
+    q, k: float32 [T, (H / heads_per_group) dk] (head h reads group h // heads_per_group), v, out: float32 [T, H dv],
+    a, b: float32 [T, H]; all may be strided views.  A_log, a_bias: [H] of one element type.
+
+    block_len > 0 (with max_new, the most rows any sequence brings): every sequence's rows are cut into blocks of
+    block_len tokens that are walked side by side, each from zeros and with its transition matrix; two kernels then carry
+    the state from block to block and add each block's incoming state to its tokens' outputs.  The same values up to
+    rounding; for long prompts."""
+    T = q.shape[0]
+    for t, n in ((q, n_heads // heads_per_group * dk), (k, n_heads // heads_per_group * dk), (v, n_heads * dv),
+                 (out, n_heads * dv), (a, n_heads), (b, n_heads)):
+        assert t.dtype == torch.float32 and (t.stride(1) == 1 or n == 1) and tuple(t.shape) == (T, n)
+    assert state.dtype == torch.float32 and state.stride(1) == 1 and state.shape[1] >= n_heads * dk * dv
+    assert A_log.numel() == a_bias.numel() == n_heads and A_log.dtype == a_bias.dtype
+    n_blocks, qp, s_loc, m_loc, kernels = 0, None, None, None, 1
+    if block_len > 0:
+        assert max_new > 0
+        n_blocks = (max_new + block_len - 1) // block_len
+        qp = torch.empty(T, n_heads * dk, dtype=torch.float32, device=q.device)
+        s_loc = torch.empty(n_seqs * n_blocks, n_heads * dk * dv, dtype=torch.float32, device=q.device)
+        m_loc = torch.empty(n_seqs * n_blocks, n_heads * dk * dk, dtype=torch.float32, device=q.device)
+        kernels = 3
+    _check(_fn("delta_rule", "odin_delta_rule")(
+        _ptr(q), c_longlong(q.stride(0)), _ptr(k), c_longlong(k.stride(0)), _ptr(v), c_longlong(v.stride(0)),
+        _ptr(a), c_longlong(a.stride(0)), _ptr(b), c_longlong(b.stride(0)), _ptr(A_log), _ptr(a_bias),
+        c_int(dtype_code(A_log.dtype)), _ptr(out), c_longlong(out.stride(0)), _ptr(state), c_longlong(state.stride(0)),
+        _ptr(seq_start), _ptr(seq_slots), c_int(n_seqs), c_int(n_heads), c_int(dk), c_int(dv), c_int(heads_per_group),
+        c_float(q_scale), c_float(unit_eps), c_int(block_len), c_int(n_blocks), _ptr(qp), _ptr(s_loc), _ptr(m_loc),
+        _stream()), "delta_rule", kernels=kernels)
 
 
 def causal_conv(src: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | None, silu: bool, state: torch.Tensor,
@@ -689,15 +751,15 @@ def latent_prep(down: torch.Tensor, q_rank: int, kv_rank: int, rot: int, pairs: 
                 tok_pos: torch.Tensor, tok_seq: torch.Tensor, block_table: torch.Tensor, cache: torch.Tensor | None,
                 write_cache: bool = True) -> None:
     """A row of the fused down projection, down = [T, q_rank + kv_rank + rot] (or float32 partial sums [parts, T, ...]),
-    is [query latent | key/value latent | key part that is rotated]: cq [T, q_rank] = RMSNorm(query latent) * q_norm;
+    is [query latent | key/value latent | key part that is rotated] (views of wider rows are fine): cq [T, q_rank] = RMSNorm(query latent) * q_norm;
     the cache row of the token's position, [kv_rank + rot] wide, becomes [RMSNorm(key/value latent) * c_norm | the key
     part rotated by the position] (pairs: elements 2i with 2i + 1, else i with i + rot / 2).
     cache: [pages, 1, PAGE, kv_rank + rot] of cq's type; cos, sin: float32 [positions, rot / 2]."""
     n = q_rank + kv_rank + rot
     if down.dim() == 3:
         n_split, T = down.shape[0], down.shape[1]
-        assert down.is_contiguous() and down.shape[2] == n
-        split_stride, row_stride = T * n, n
+        assert down.stride(2) == 1 and down.shape[2] == n
+        split_stride, row_stride = down.stride(0), down.stride(1)
     else:
         n_split, T, split_stride, row_stride = 1, down.shape[0], 0, down.stride(0)
         assert down.stride(1) == 1 and down.shape[1] == n
@@ -718,17 +780,33 @@ def latent_prep(down: torch.Tensor, q_rank: int, kv_rank: int, rot: int, pairs: 
         c_int(PAGE), c_int(1 if write_cache else 0), _stream()), "latent_prep")
 
 
-def heads_linear(a: torch.Tensor, a_head_stride: int, w: torch.Tensor, out: torch.Tensor, out_head_stride: int) -> None:
+def _parts_view(t: torch.Tensor) -> tuple[int, int, int]:
+    """(parts, their distance, row stride) of a product's output or a view of its columns: [T, n] or [parts, T, n]."""
+    assert t.stride(-1) == 1 or t.shape[-1] == 1
+    return (t.shape[0], t.stride(0), t.stride(1)) if t.dim() == 3 else (1, 0, t.stride(0))
+
+
+def heads_linear(a: torch.Tensor, a_head_stride: int, w: torch.Tensor, out: torch.Tensor, out_head_stride: int,
+                 gate: torch.Tensor | None = None) -> None:
     """A product per head: out[t, h * out_head_stride + n] = sum_k a[t, h * a_head_stride + k] * w[h, k, n] for
-    w [H, K, N] (input channel before output channel); a and out may be views with any row stride."""
+    w [H, K, N] (input channel before output channel); a and out may be views with any row stride, a also float32 partial
+    sums [parts, T, ...] of a split product.  gate ([T, H], a view or partial sums): head h's outputs are multiplied by
+    sigmoid(gate[t, h])."""
     H, K, N = w.shape
-    T = a.shape[0]
-    assert w.is_contiguous() and a.stride(1) == 1 and out.stride(1) == 1 and out.shape[0] == T
-    assert a.shape[1] >= (H - 1) * a_head_stride + K and out.shape[1] >= (H - 1) * out_head_stride + N
+    T = a.shape[-2]
+    assert w.is_contiguous() and a.stride(-1) == 1 and out.stride(1) == 1 and out.shape[0] == T
+    assert a.shape[-1] >= (H - 1) * a_head_stride + K and out.shape[1] >= (H - 1) * out_head_stride + N
+    a_split, a_ss, a_rs = _parts_view(a)
+    g_split, g_ss, g_rs = (1, 0, 0)
+    if gate is not None:
+        assert tuple(gate.shape[-2:]) == (T, H)
+        g_split, g_ss, g_rs = _parts_view(gate)
     _check(_fn("latent", "odin_heads_linear")(
-        _ptr(a), c_int(dtype_code(a.dtype)), c_longlong(a.stride(0)), c_longlong(a_head_stride), _ptr(w),
-        c_int(dtype_code(w.dtype)), _ptr(out), c_int(dtype_code(out.dtype)), c_longlong(out.stride(0)),
-        c_longlong(out_head_stride), c_int(T), c_int(H), c_int(N), c_int(K), _stream()), "heads_linear")
+        _ptr(a), c_int(dtype_code(a.dtype)), c_int(a_split), c_longlong(a_ss), c_longlong(a_rs), c_longlong(a_head_stride),
+        _ptr(w), c_int(dtype_code(w.dtype)), _ptr(out), c_int(dtype_code(out.dtype)), c_longlong(out.stride(0)),
+        c_longlong(out_head_stride), c_int(T), c_int(H), c_int(N), c_int(K), _ptr(gate),
+        c_int(dtype_code(gate.dtype) if gate is not None else 0), c_int(g_split), c_longlong(g_ss), c_longlong(g_rs),
+        _stream()), "heads_linear")
 
 
 def rope_heads(src: torch.Tensor, src_head_stride: int, dst: torch.Tensor, dst_head_stride: int, n_heads: int, width: int,
@@ -900,7 +978,8 @@ def head_prep(qkv: torch.Tensor, n_q: int, n_kv: int, head_dim: int, q_norm: tor
               tok_pos: torch.Tensor, tok_seq: torch.Tensor, block_table: torch.Tensor,
               k_cache: torch.Tensor | None, v_cache: torch.Tensor | None, write_kv: bool = True,
               q_out: torch.Tensor | None = None, bias: torch.Tensor | None = None, unit_norm_after: bool = False,
-              v_head_dim: int | None = None, whole_norm: bool = False, pairs: bool = False) -> torch.Tensor:
+              v_head_dim: int | None = None, whole_norm: bool = False, pairs: bool = False,
+              v_first: torch.Tensor | None = None, v_lambda: float = 0.0, v_keep: torch.Tensor | None = None) -> torch.Tensor:
     """Per-head RMSNorm and rotation of q and k, and the cache write of k and v.
 
     bias: one value per column of the projection, added first.  unit_norm_after: instead of the
@@ -908,6 +987,8 @@ def head_prep(qkv: torch.Tensor, n_q: int, n_kv: int, head_dim: int, q_norm: tor
     (q_norm and k_norm are then None).  v_head_dim: size of a value head when it differs from head_dim.
     whole_norm: the norm before the rotation runs over the token's whole q projection at once (and its whole k projection),
     with q_norm [n_q head_dim] and k_norm [n_kv head_dim].  pairs: the rotation pairs element 2i with 2i + 1.
+    v_first ([T, n_kv v_head_dim] of the cache's type): what is cached is (1 - v_lambda) v + v_lambda v_first; v_keep (the
+    same shape): takes this projection's own values.
 
     qkv: [T, (n_q + 2 n_kv) head_dim], or float32 partial sums [parts, T, ...] of a split
     product (added first).  q goes to q_out ([T, n_q head_dim], of the cache's type); without
@@ -942,6 +1023,9 @@ def head_prep(qkv: torch.Tensor, n_q: int, n_kv: int, head_dim: int, q_norm: tor
         assert k_cache.is_contiguous() and v_cache.is_contiguous()
         assert tuple(k_cache.shape[1:]) == (n_kv, PAGE, head_dim), "cache layout is [page][kv head][64][hd]"
         assert tuple(v_cache.shape[1:]) == (n_kv, PAGE, vd), "value cache layout is [page][kv head][64][vd]"
+    for v in (v_first, v_keep):
+        if v is not None:
+            assert v.is_contiguous() and tuple(v.shape) == (T, n_kv * vd) and v.dtype == q_out.dtype and write_kv
     _check(_fn("head_prep", "odin_head_prep")(
         _ptr(qkv), c_int(dtype_code(qkv.dtype)), c_int(n_split), c_longlong(split_stride), _ptr(q_out),
         c_longlong(q_out.stride(0)), c_int(dtype_code(q_out.dtype)), c_int(T), c_int(n_q), c_int(n_kv),
@@ -951,7 +1035,8 @@ def head_prep(qkv: torch.Tensor, n_q: int, n_kv: int, head_dim: int, q_norm: tor
         c_float(eps),
         _ptr(cos), _ptr(sin), c_int(rotary_dim), c_int(cos.shape[0]), _ptr(tok_pos), _ptr(tok_seq),
         _ptr(block_table), c_int(block_table.stride(0)), _ptr(k_cache), _ptr(v_cache), c_int(PAGE),
-        c_int(1 if write_kv else 0), c_int(1 if pairs else 0), _stream()), "head_prep")
+        c_int(1 if write_kv else 0), c_int(1 if pairs else 0), _ptr(v_first), _ptr(v_keep), c_float(v_lambda), _stream()),
+        "head_prep")
     return q_out
 
 

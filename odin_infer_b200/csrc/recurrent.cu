@@ -15,7 +15,7 @@
 // step to step; a sequence's tokens are walked in order by one CTA per (sequence, head), column j of S
 // held in the registers of four lanes, so the result does not depend on how the tokens were cut into
 // steps or on what else is in the batch.  Decays, gates, exponentials and the state are 32-bit.
-#include "common.cuh"
+#include "recurrence_blocks.cuh"
 
 // ------------------------------------------------------------ token shift
 // out[s][t][:] = h[t] + (prev - h[t]) * mu[s], s < n_mix.  Rows of sequence -1 are skipped.
@@ -81,36 +81,6 @@ extern "C" int odin_token_shift(const void* h, int dtype, const float* state, lo
 #define REC_GLA 3     // w = sigmoid(raw + c0)^c1 = exp(c1 logsigmoid(raw + c0)); S = diag(w) S + k v^T; o = S^T (q_scale q)
 #define REC_SSD 4     // per head and token one step dt = softplus(raw[head] + c1[head]) and one decay w = exp(-exp(c0[head]) dt);
                       // S = w S + (dt k) v^T; o = S^T q; q and k belong to the head's group (heads_per_group heads share them)
-// Threads that share a column of S: each owns a quarter of the key channels.  (Sixteen lanes per column, a quarter of
-// the registers each, walked a prompt of 2,048 tokens a fifth faster and made a decode step three to four times slower:
-// four times the threads for the same work.)
-#define REC_SPLIT 4
-#define REC_MAX_DK 256
-
-struct RecParams {
-    const float* q; long long q_stride;   // [rows, H*dk] projections (32-bit), row strides in elements
-    const float* k; long long k_stride;   // REC_BONUS and REC_FIXED
-    const float* g; long long g_stride;   // the raw decay / forget gate (REC_FIXED: unused)
-    const float* v; long long v_stride;   // [rows, H*dv]
-    VecRef c0, c1;                        // per (head, key channel): REC_BONUS w0 and u; REC_GATED bias and lower bound; REC_FIXED: c0 per head
-    float* o; long long o_stride;         // [rows, H*dv]
-    float* state; long long state_stride; // per slot: [H][dk][dv] floats
-    const int* seq_start; const int* seq_slots;
-    int H, dk, dv;
-    float q_scale;        // REC_GLA: factor on q
-    int heads_per_group;  // REC_SSD: heads that share one q and one k (their columns: group * dk)
-    // the token shift's memory: after the step the sequence's last row of h goes to its state
-    const void* shift_src; int shift_is_bf16; float* shift_state; long long shift_stride; int width;
-    // Blocks of tokens (block_len > 0): a CTA walks one block of one sequence from a state of zeros and leaves
-    // the block's own state in s_loc, the product of the block's decays per key channel in d_tot, and per token
-    // q times the decays since the block's start in qp; two small kernels then carry the state from block to block
-    // and add what each block's incoming state contributes to its tokens' outputs.
-    int block_len, n_blocks;
-    float* qp;     // [rows, H*dk]
-    float* s_loc;  // [sequences * n_blocks][H][dk][dv]
-    float* d_tot;  // [sequences * n_blocks][H*dk]
-};
-
 // One CTA per (sequence, head) walks the sequence's tokens in order.  Column j of S belongs to REC_SPLIT lanes of
 // one warp (lane = part * 8 + j % 8), each holding SL consecutive key channels of it in registers; a token costs
 // each thread SL multiply-adds for the output and SL for the state, and the column's output is the sum of its
@@ -122,8 +92,6 @@ struct RecParams {
 // has more than 512 threads and the state fits the registers; the launcher takes fewer columns per CTA when there
 // are few (sequence, head) pairs, so that a long prompt of one sequence still occupies the GPU.  A column's
 // arithmetic does not depend on which CTA holds it.
-#define REC_COLS 128
-#define REC_FETCH 4   // elements of each input that a thread fetches ahead per block of tokens
 template <int SL, int MODE, bool BLOCKS>
 __global__ void __launch_bounds__(REC_COLS * REC_SPLIT)
 linear_recurrence_kernel(RecParams p) {
@@ -345,88 +313,6 @@ recurrence_carry_kernel(RecParams p) {
     *st = S;
 }
 
-// o[t, head, :] += (q_t * decays since the block's start)^T S_in(block): 64 (or 32) tokens by 32 columns per CTA pass.
-// Shared memory: the incoming state's 32 columns [dk][32], then (dk a multiple of four) 64 tokens' q [64][dk], which the
-// CTA fetches with loads that all go out together; a warp then takes eight tokens and reads four channels of a token's q
-// in one broadcast.  Every sum runs over the channels in their order, whichever path computes it.
-#define CARRY_OUT_TOK 64
-__global__ void __launch_bounds__(256)
-recurrence_carry_out_kernel(RecParams p) {
-    extern __shared__ __align__(16) float co_smem[];
-    float (*tile)[32] = reinterpret_cast<float (*)[32]>(co_smem);
-    float* qsm = co_smem + (size_t)p.dk * 32;
-    pdl_trigger();
-    const int item = blockIdx.x, head = blockIdx.y;
-    const int b = item / p.n_blocks;
-    const int lane = threadIdx.x & 31, lane_t = threadIdx.x >> 5;
-    const int col = blockIdx.z * 32 + lane;
-    const int seq_end = p.seq_start[b + 1];
-    const int row0 = p.seq_start[b] + (item % p.n_blocks) * p.block_len;
-    const int row1 = min(seq_end, row0 + p.block_len);
-    pdl_wait();
-    if (row1 <= row0) return;
-    const float* sin = p.s_loc + ((size_t)item * p.H + head) * p.dk * p.dv;
-    for (int e = threadIdx.x; e < p.dk * 32; e += blockDim.x) {
-        const int i = e >> 5, c = blockIdx.z * 32 + (e & 31);
-        tile[i][e & 31] = c < p.dv ? sin[(size_t)i * p.dv + c] : 0.f;
-    }
-    const size_t qs = (size_t)p.H * p.dk;
-    if ((p.dk & 3) == 0) {
-        const int dk4 = p.dk >> 2;
-        for (int tb = row0; tb < row1; tb += CARRY_OUT_TOK) {
-            __syncthreads();   // the pass before has read its q (and, the first time, the tile is there after the next one)
-            for (int e = threadIdx.x; e < CARRY_OUT_TOK * dk4; e += blockDim.x) {
-                const int u = e / dk4, c4 = e % dk4;
-                if (tb + u < row1)
-                    reinterpret_cast<float4*>(qsm)[e] =
-                        __ldg(reinterpret_cast<const float4*>(p.qp + (size_t)(tb + u) * qs + (size_t)head * p.dk) + c4);
-            }
-            __syncthreads();
-            const int t0 = tb + lane_t * 8;
-            const int nt = min(8, row1 - t0);
-            if (nt <= 0) continue;
-            float acc[8];
-#pragma unroll
-            for (int u = 0; u < 8; ++u) acc[u] = 0.f;
-            const float* qw = qsm + (size_t)lane_t * 8 * p.dk;
-            for (int i = 0; i < p.dk; i += 4) {
-                const float s0 = tile[i][lane], s1 = tile[i + 1][lane], s2 = tile[i + 2][lane], s3 = tile[i + 3][lane];
-#pragma unroll
-                for (int u = 0; u < 8; ++u)
-                    if (u < nt) {
-                        const float4 q4 = *reinterpret_cast<const float4*>(qw + u * p.dk + i);
-                        acc[u] = fmaf(q4.x, s0, acc[u]);
-                        acc[u] = fmaf(q4.y, s1, acc[u]);
-                        acc[u] = fmaf(q4.z, s2, acc[u]);
-                        acc[u] = fmaf(q4.w, s3, acc[u]);
-                    }
-            }
-            if (col < p.dv) {
-#pragma unroll
-                for (int u = 0; u < 8; ++u)
-                    if (u < nt) p.o[(size_t)(t0 + u) * p.o_stride + (size_t)head * p.dv + col] += acc[u];
-            }
-        }
-        return;
-    }
-    __syncthreads();
-    for (int t0 = row0 + lane_t * 4; t0 < row1; t0 += 32) {   // a warp takes four tokens at a time
-        float acc[4] = {0.f, 0.f, 0.f, 0.f};
-        const float* qrow = p.qp + (size_t)t0 * qs + (size_t)head * p.dk;
-        for (int i = 0; i < p.dk; ++i) {
-            const float sv = tile[i][lane];
-#pragma unroll
-            for (int u = 0; u < 4; ++u)
-                if (t0 + u < row1) acc[u] = fmaf(__ldg(qrow + u * qs + i), sv, acc[u]);
-        }
-        if (col < p.dv) {
-#pragma unroll
-            for (int u = 0; u < 4; ++u)
-                if (t0 + u < row1) p.o[(size_t)(t0 + u) * p.o_stride + (size_t)head * p.dv + col] += acc[u];
-        }
-    }
-}
-
 extern "C" int odin_linear_recurrence(int mode, const float* q, long long q_stride, const float* k, long long k_stride,
                                       const float* g, long long g_stride, const float* v, long long v_stride,
                                       const void* c0, const void* c1, int c_dtype, float* o, long long o_stride,
@@ -491,13 +377,8 @@ extern "C" int odin_linear_recurrence(int mode, const float* q, long long q_stri
     if (blocks) {
         odin_launch(recurrence_carry_kernel, dim3(n_seqs, H, (dk * dv + 255) / 256), dim3(256), 0, s, p);
         ODIN_LAUNCH_CHECK();
-        const size_t co_smem = (size_t)dk * 32 * sizeof(float) + ((dk & 3) == 0 ? (size_t)CARRY_OUT_TOK * dk * sizeof(float) : 0);
-        if (co_smem > 48 * 1024) {
-            cudaError_t e = cudaFuncSetAttribute(recurrence_carry_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)co_smem);
-            if (e != cudaSuccess) return (int)e;
-        }
-        odin_launch(recurrence_carry_out_kernel, dim3(n_items, H, (dv + 31) / 32), dim3(256), co_smem, s, p);
-        ODIN_LAUNCH_CHECK();
+        const int rc = launch_recurrence_carry_out(p, n_items, s);
+        if (rc != 0) return rc;
     }
     return 0;
 }

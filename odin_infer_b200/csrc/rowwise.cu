@@ -558,7 +558,9 @@ extern "C" int odin_softcap(float* z, long long stride, int rows, int n, float c
 
 // ------------------------------------------------------------ several terms into one update, normed, added, normed again
 // y = sum_i scale_i * rowscale_i[r] * f_i(sum of term i's parts), f_i the identity or w_i * v / rms(v) over the row;
-// then x[r] += post_w * y / rms(y) (post_w null: x[r] += y), and out = next_w * x[r] / rms(x[r]) (next_w null: no output).
+// then x[r] += post_w * y / rms(y) (post_w null: x[r] += y), and out = next_w * x[r] / rms(x[r]) (next_w null: out = x[r]
+// converted, or no output at all).  Either of these two norms may be a layer norm (`center`): the row's mean is taken off
+// first, the variance is the mean of the squared deviations, and a bias may follow the weight.
 // Without x the sum itself goes to out as 32-bit values.  rows: gather these rows (x is then left as it is).
 // One CTA per row; every sum runs in an order that the width and the block size fix.
 #define COMBINE_MAX_TERMS 4
@@ -567,11 +569,12 @@ struct CombineTerm {
     float scale; const float* row_scale; VecRef norm_w; float norm_eps;
 };
 struct CombineArgs { CombineTerm t[COMBINE_MAX_TERMS]; int n; };
+struct CombineNorm { VecRef w, b; float eps; int center; };   // w null: no norm
 
 template <typename TO, bool VEC>
 __global__ void __launch_bounds__(ROW_THREADS)
-combine_add_kernel(float* __restrict__ x, CombineArgs a, VecRef post_w, float post_eps, VecRef next_w, float next_eps,
-                   TO* __restrict__ out, const int* __restrict__ rows, const int* __restrict__ tok_seq, int d) {
+combine_add_kernel(float* __restrict__ x, CombineArgs a, CombineNorm post, CombineNorm next, TO* __restrict__ out,
+                   const int* __restrict__ rows, const int* __restrict__ tok_seq, int d) {
     __shared__ float red[32];
     extern __shared__ __align__(16) float cbuf[];
     float* acc = cbuf;        // d
@@ -595,6 +598,11 @@ combine_add_kernel(float* __restrict__ x, CombineArgs a, VecRef post_w, float po
         if (VEC) { const float4 q = w.at4(j); v[0] = q.x; v[1] = q.y; v[2] = q.z; v[3] = q.w; }
         else v[0] = w.at(j);
     };
+    if (a.n == 0)
+        for (int j = j0; j < d; j += dj) {
+#pragma unroll
+            for (int e = 0; e < W; ++e) acc[j + e] = 0.f;
+        }
     for (int i = 0; i < a.n; ++i) {
         const CombineTerm& tm = a.t[i];
         float ss = 0.f;
@@ -636,29 +644,47 @@ combine_add_kernel(float* __restrict__ x, CombineArgs a, VecRef post_w, float po
         }
         return;
     }
-    float rs = 1.0f;
-    if (post_w.p != nullptr) {
-        float ss = 0.f;
+    // (mean, 1 / root) of a row that the threads hold in `buf`; without `center` the mean is zero
+    auto statistics = [&](const float* buf, const CombineNorm& nm, float sum, float sum_sq, float& mean, float& rs) {
+        mean = 0.f;
+        if (nm.center) {
+            mean = block_sum(sum, red) / (float)d;
+            sum_sq = 0.f;
+            for (int j = j0; j < d; j += dj) {
+#pragma unroll
+                for (int e = 0; e < W; ++e) { const float c = buf[j + e] - mean; sum_sq += c * c; }
+            }
+        }
+        float ss = block_sum(sum_sq, red);
+        ss /= (float)d;
+        ss += nm.eps;
+        rs = 1.0f / sqrtf(ss);
+    };
+    float mean = 0.f, rs = 1.0f;
+    if (post.w.p != nullptr) {
+        float s1 = 0.f, ss = 0.f;
         for (int j = j0; j < d; j += dj) {
 #pragma unroll
-            for (int e = 0; e < W; ++e) ss += acc[j + e] * acc[j + e];
+            for (int e = 0; e < W; ++e) { s1 += acc[j + e]; ss += acc[j + e] * acc[j + e]; }
         }
-        ss = block_sum(ss, red);
-        ss /= (float)d;
-        ss += post_eps;
-        rs = 1.0f / sqrtf(ss);
+        statistics(acc, post, s1, ss, mean, rs);
     }
     float* xr = x + (size_t)r * d;
-    float s2 = 0.f;
+    float s1 = 0.f, s2 = 0.f;
     for (int j = j0; j < d; j += dj) {
-        float xv[W], w[W];
+        float xv[W], w[W], b[W];
         if (VEC) { const float4 q = ld4(xr + j); xv[0] = q.x; xv[1] = q.y; xv[2] = q.z; xv[3] = q.w; }
         else xv[0] = xr[j];
-        if (post_w.p != nullptr) weights(post_w, j, w);
+        if (post.w.p != nullptr) weights(post.w, j, w);
+        if (post.b.p != nullptr) weights(post.b, j, b);
 #pragma unroll
         for (int e = 0; e < W; ++e) {
-            xv[e] += post_w.p != nullptr ? w[e] * (rs * acc[j + e]) : acc[j + e];
+            float u = acc[j + e];
+            if (post.w.p != nullptr) u = w[e] * (rs * (u - mean));
+            if (post.b.p != nullptr) u += b[e];
+            xv[e] += u;
             tmp[j + e] = xv[e];
+            s1 += xv[e];
             s2 += xv[e] * xv[e];
         }
         if (rows == nullptr) {
@@ -666,26 +692,31 @@ combine_add_kernel(float* __restrict__ x, CombineArgs a, VecRef post_w, float po
             else xr[j] = xv[0];
         }
     }
-    if (next_w.p == nullptr) return;
-    s2 = block_sum(s2, red);
-    s2 /= (float)d;
-    s2 += next_eps;
-    const float r2 = 1.0f / sqrtf(s2);
+    if (out == nullptr) return;
+    float mean2 = 0.f, r2 = 1.0f;
+    if (next.w.p != nullptr) statistics(tmp, next, s1, s2, mean2, r2);
     TO* orow = out + (size_t)blockIdx.x * d;
     for (int j = j0; j < d; j += dj) {
-        float w[W];
-        weights(next_w, j, w);
-        if (VEC) st4(orow + j, make_float4(w[0] * (r2 * tmp[j]), w[1] * (r2 * tmp[j + 1]), w[2] * (r2 * tmp[j + 2]), w[3] * (r2 * tmp[j + 3])));
-        else orow[j] = from_f32<TO>(w[0] * (r2 * tmp[j]));
+        float v[W], w[W], b[W];
+        if (next.w.p != nullptr) weights(next.w, j, w);
+        if (next.b.p != nullptr) weights(next.b, j, b);
+#pragma unroll
+        for (int e = 0; e < W; ++e) {
+            v[e] = next.w.p != nullptr ? w[e] * (r2 * (tmp[j + e] - mean2)) : tmp[j + e];
+            if (next.b.p != nullptr) v[e] += b[e];
+        }
+        if (VEC) st4(orow + j, make_float4(v[0], v[VEC ? 1 : 0], v[VEC ? 2 : 0], v[VEC ? 3 : 0]));
+        else orow[j] = from_f32<TO>(v[0]);
     }
 }
 
 extern "C" int odin_combine_add(float* x, int n_terms, const void* const* ptrs, const int* dtypes, const int* n_splits,
                                 const long long* split_strides, const float* scales, const float* const* row_scales,
                                 const void* const* norm_ws, const int* norm_w_dtypes, const float* norm_eps,
-                                const void* post_w, int post_w_dtype, float post_eps, const void* next_w, int next_w_dtype,
-                                float next_eps, void* out, int out_dtype, const int* rows, const int* tok_seq, int n_rows,
-                                int d, void* stream) {
+                                const void* post_w, int post_w_dtype, const void* post_b, int post_b_dtype, float post_eps,
+                                int post_center, const void* next_w, int next_w_dtype, const void* next_b, int next_b_dtype,
+                                float next_eps, int next_center, void* out, int out_dtype, const int* rows,
+                                const int* tok_seq, int n_rows, int d, void* stream) {
     if (n_rows <= 0) return 0;
     if (n_terms < 0 || n_terms > COMBINE_MAX_TERMS || d <= 0) return ODIN_ERR_BAD_ARG;
     if (x == nullptr && (out == nullptr || out_dtype != ODIN_F32)) return ODIN_ERR_BAD_ARG;
@@ -702,10 +733,11 @@ extern "C" int odin_combine_add(float* x, int n_terms, const void* const* ptrs, 
         a.t[i].norm_w = VecRef{norm_ws[i], norm_w_dtypes[i] == ODIN_BF16}; a.t[i].norm_eps = norm_eps[i];
         all_bits |= (uintptr_t)ptrs[i] | (uintptr_t)norm_ws[i] | (uintptr_t)(split_strides[i] * 4);
     }
-    all_bits |= (uintptr_t)x | (uintptr_t)out | (uintptr_t)post_w | (uintptr_t)next_w;
+    all_bits |= (uintptr_t)x | (uintptr_t)out | (uintptr_t)post_w | (uintptr_t)next_w | (uintptr_t)post_b | (uintptr_t)next_b;
     const bool vec = (d % 4 == 0) && (all_bits % 16 == 0);
     cudaStream_t s = (cudaStream_t)stream;
-    VecRef pw{post_w, post_w_dtype == ODIN_BF16}, nw{next_w, next_w_dtype == ODIN_BF16};
+    const CombineNorm post{VecRef{post_w, post_w_dtype == ODIN_BF16}, VecRef{post_b, post_b_dtype == ODIN_BF16}, post_eps, post_center};
+    const CombineNorm next{VecRef{next_w, next_w_dtype == ODIN_BF16}, VecRef{next_b, next_b_dtype == ODIN_BF16}, next_eps, next_center};
 #define GO(TO)                                                                                                       \
     do {                                                                                                             \
         auto kern = vec ? combine_add_kernel<TO, true> : combine_add_kernel<TO, false>;                              \
@@ -713,8 +745,7 @@ extern "C" int odin_combine_add(float* x, int n_terms, const void* const* ptrs, 
             cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);       \
             if (e != cudaSuccess) return (int)e;                                                                     \
         }                                                                                                            \
-        odin_launch(kern, dim3(n_rows), dim3(ROW_THREADS), smem, s, x, a, pw, post_eps, nw, next_eps, (TO*)out, rows,   \
-                    tok_seq, d);                                                                                     \
+        odin_launch(kern, dim3(n_rows), dim3(ROW_THREADS), smem, s, x, a, post, next, (TO*)out, rows, tok_seq, d);  \
     } while (0)
     if (out == nullptr || out_dtype == ODIN_F32) GO(float);
     else if (out_dtype == ODIN_BF16) GO(bf16);

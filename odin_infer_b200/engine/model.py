@@ -98,12 +98,14 @@ class DecoderModel:
 
     def forward(self, rt, step) -> torch.Tensor | None:
         """Runs the step's tokens; returns 32-bit logits [wanted rows, vocab] (None if none wanted)."""
+        step.carried = {}   # what a layer hands to later layers of the same step
         x = self.embedding.forward(rt, step)
         for pe in self.position_encodings.values():
             pe.on_embedding(rt, step, x)
         pending = None
         for idx, e in enumerate(self.spec.schedule):
             x, pending = self.layers[e.layer].forward(rt, step, x, pending, idx)
+        step.carried = {}
         if step.n_logit_rows == 0:
             return None
         delta, bias = split_update(pending)

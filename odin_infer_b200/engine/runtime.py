@@ -225,13 +225,15 @@ class Runtime:
 
     # ---- experts chosen per token ----------------------------------------
     def experts(self, h: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor,
-                wts: torch.Tensor, activation: str, gated: bool = True) -> torch.Tensor:
+                wts: torch.Tensor, activation: str, gated: bool = True, weigh_input: bool = False) -> torch.Tensor:
         """The chosen experts' gated feed-forwards for every (token, choice): ids / wts [T, per] name each
         choice's expert (-1: none) and weight; w_gate_up [experts, 2 inner, width], w_down [experts, width,
         inner].  Returns the tokens' update: float32 [per, T, width] partial sums (slice k holds every token's
         k-th choice, weighted) from the row-by-row kernels, or float32 [T, width] from the grouped products.
-        gated=False: an expert is W_down act(W_up h) and w_gate_up is [experts, inner, width]."""
+        gated=False: an expert is W_down act(W_up h) and w_gate_up is [experts, inner, width].
+        weigh_input: the weight multiplies what the expert reads instead of what it answers."""
         T, per = ids.shape
+        in_wts, out_wts = (wts, None) if weigh_input else (None, wts)
         inner, width = w_down.shape[2], w_down.shape[1]
         if T * per >= MOE_GROUPED_FROM_ROWS and ops.moe_grouped_supported(h, w_gate_up, w_down) and width % 4 == 0:
             # many rows: sorted by expert and multiplied tile by tile on the tensor cores (a row's weights are read
@@ -243,18 +245,18 @@ class Runtime:
             tile_expert = self.empty(places // 128, dtype=torch.int32)
             ops.moe_plan(ids, n_e, place_of_row, row_of_place, tile_expert)
             hs = self.empty(places, h.shape[1])
-            ops.moe_gather(h, row_of_place, per, hs)
+            ops.moe_gather(h, row_of_place, per, hs, in_wts)
             a = self.empty(places, inner)
             ops.moe_grouped(hs, w_gate_up, tile_expert, a, activation, gated=gated)   # the activation rides in the epilogue
             c = self.empty(places, width, dtype=torch.float32)
             ops.moe_grouped(a, w_down, tile_expert, c)
             y = self.empty(T, width, dtype=torch.float32)
-            ops.moe_combine(c, place_of_row, wts, y)
+            ops.moe_combine(c, place_of_row, out_wts, y)
             return y
         a = self.empty(T * per, inner)
-        ops.moe_gate_up(h, w_gate_up, ids, activation, a, gated=gated)
+        ops.moe_gate_up(h, w_gate_up, ids, activation, a, gated=gated, in_wts=in_wts)
         y = self.empty(per, T, width, dtype=torch.float32)
-        ops.moe_down(a, w_down, ids, wts, y)
+        ops.moe_down(a, w_down, ids, out_wts, y)
         return y
 
     # ---- attention over the cache ---------------------------------------

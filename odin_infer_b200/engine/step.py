@@ -42,13 +42,17 @@ class StepBatch:
     (first token row; n_seqs + 1 entries), seq_len_after[b] (its length once this step
     is done), and one block table row per cache group.  logit_rows: the token rows
     whose logits are wanted.  Host copies for parts that size their launches:
-    n_seqs, n_tokens, slots, lengths_after, seq_start_host, all_single, max_new.
+    n_seqs, n_tokens, slots, lengths_after, seq_start_host, all_single, max_new.  carried: device
+    tensors by name that a layer hands to later layers of the same step.
     """
+
+    carried: dict
 
     def __init__(self, cache, entries: list[StepEntry], start_positions: list[int], device,
                  pad_rows_to: int = 0, pad_seqs_to: int = 0, all_rows_wanted: bool = False):
         self.cache = cache
         self.device = device
+        self.carried = {}
         self.n_seq_cap = max(len(entries), pad_seqs_to)
         self.n_row_cap = max(sum(len(e.tokens) for e in entries), pad_rows_to)
         self.all_rows_wanted = all_rows_wanted

@@ -32,6 +32,9 @@ class GQAttention(Mixer):
     denominator (no key, no value, not scaled).  gate: name of a matrix G; the heads' outputs are multiplied by
     sigmoid(G h) before the output projection, one factor per element (G: [n_q_heads * v_head_dim, width]) or,
     with gate_per_head, one per head (G: [n_q_heads, width]); G is fused with q, k and v into one product.
+    value_mix = {"key": str, "lambda": name of a scalar tensor or None}: values are mixed with those of an earlier layer of
+    the same step.  Without a "lambda" this mixer's own values are kept under `key` for the layers after it; with one, what
+    it attends over (and caches) is (1 - lambda) v + lambda v_kept.
     """
 
     graph_safe = True
@@ -41,7 +44,7 @@ class GQAttention(Mixer):
                  position_encoding: str | None = None, qk_norm=True, eps: float = 1e-6,
                  window: int = 0, kv_shared: bool = False, chunk: int = 0, biases: dict | None = None,
                  scale: float = 0.0, softcap: float = 0.0, v_head_dim: int = 0, sink: str | None = None,
-                 gate: str | None = None, gate_per_head: bool = False):
+                 gate: str | None = None, gate_per_head: bool = False, value_mix: dict | None = None):
         if n_q_heads % n_kv_heads:
             raise ValueError(f"{n_q_heads} query heads are not a multiple of {n_kv_heads} kv heads")
         if qk_norm not in (True, False, "unit_after", "whole"):
@@ -59,7 +62,12 @@ class GQAttention(Mixer):
         self.n_gate = 0 if gate is None else (self.n_q if self.gate_per_head else self.n_q * self.vd)
         self.plain_heads = (self.bias_names is None and not self.unit_after and not self.whole_norm and self.vd == self.hd
                             and self.chunk == 0 and self.scale == 0.0 and self.softcap == 0.0
-                            and sink is None and gate is None)
+                            and sink is None and gate is None and value_mix is None)
+        if value_mix is not None and kv_shared:
+            raise ValueError("a mixer without values of its own cannot mix them")
+        self.mix_key = None if value_mix is None else str(value_mix["key"])
+        self.mix_name = None if value_mix is None else value_mix.get("lambda")
+        self.mix_lambda = 0.0
         self.sink = None
         self.pe = None          # set by the model from pe_name
         self.w_qkv = self.w_o = self.q_norm = self.k_norm = self.b_qkv = self.b_o = None
@@ -83,6 +91,8 @@ class GQAttention(Mixer):
                 out += [ParamSpec(b["k"], (self.n_kv * self.hd,)), ParamSpec(b["v"], (self.n_kv * self.vd,))]
             if b.get("o"):
                 out.append(ParamSpec(b["o"], (self.width,)))
+        if self.mix_name is not None:
+            out.append(ParamSpec(self.mix_name, (), init="unit"))
         if self.sink_name is not None:
             out.append(ParamSpec(self.sink_name, (self.n_q,), init="logit"))
         if self.gate_name is not None:
@@ -102,6 +112,8 @@ class GQAttention(Mixer):
             if len({t.dtype for t in mats}) > 1:
                 mats = [t.to(torch.float32) for t in mats]
             self.w_qkv = torch.cat(mats, dim=0).contiguous()
+        if self.mix_name is not None:
+            self.mix_lambda = float(tensors[self.mix_name].to(torch.float32).item())
         if self.sink_name is not None:
             self.sink = tensors[self.sink_name].to(torch.float32).contiguous()
         self.w_o = tensors[n["o"]]
@@ -165,11 +177,17 @@ class GQAttention(Mixer):
         pairs = rot is not None and getattr(self.pe, "layout", "halves") == "pairs"
         if not self.plain_heads or pairs:
             q_out = rt.empty(T, self.n_q * self.hd)
+            mix = {}
+            if self.mix_name is not None:
+                mix = dict(v_first=step.carried[self.mix_key], v_lambda=self.mix_lambda)
+            elif self.mix_key is not None:
+                mix = dict(v_keep=rt.empty(T, self.n_kv * self.vd))
+                step.carried[self.mix_key] = mix["v_keep"]
             q = ops.head_prep(qkv, self.n_q, 0 if self.kv_shared else self.n_kv, self.hd,
                               self.q_norm if self.qk_norm else None, self.k_norm if self.qk_norm else None, self.eps,
                               cos, sin, rot_dim, step.tok_pos, step.tok_seq, block_table, k_line, v_line,
                               write_kv=writes, q_out=q_out, bias=self.b_qkv, unit_norm_after=self.unit_after,
-                              v_head_dim=self.vd, whole_norm=self.whole_norm, pairs=pairs)
+                              v_head_dim=self.vd, whole_norm=self.whole_norm, pairs=pairs, **mix)
             rt.attention(step, q, o, self.n_q, self.n_kv, self.hd, k_line, v_line, block_table, self.window,
                          chunk=self.chunk, scale=self.scale, softcap=self.softcap, v_head_dim=self.vd, sink=self.sink)
             if self.gate_name is not None:

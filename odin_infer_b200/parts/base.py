@@ -133,12 +133,12 @@ class Combined(list):
 
 
 class Normed:
-    """An update that passes an RMSNorm of its own before it is added: x += weight * u / rms(u), u the sum of `update`
-    (a tensor, `Several` or `Combined`).  Only a norm that says `takes_terms` may follow; it does the sum, this norm,
-    the add and its own norm in one kernel."""
+    """An update that passes a norm of its own before it is added: x += weight * u / rms(u), u the sum of `update`
+    (a tensor, `Several` or `Combined`); with `center` a layer norm, x += weight * (u - mean(u)) / std(u) + bias.  Only a
+    norm that says `takes_terms` may follow; it does the sum, this norm, the add and its own norm in one kernel."""
 
-    def __init__(self, update, weight: torch.Tensor, eps: float):
-        self.update, self.weight, self.eps = update, weight, float(eps)
+    def __init__(self, update, weight: torch.Tensor, eps: float, bias: torch.Tensor | None = None, center: bool = False):
+        self.update, self.weight, self.eps, self.bias, self.center = update, weight, float(eps), bias, bool(center)
 
 
 def update_factor(pending) -> float:
@@ -177,6 +177,12 @@ class Norm(Part):
     takes_several = False   # `delta` may be a list of up to three updates
     takes_scale = False     # takes a keyword `scale=`: x += scale * (the updates)
     takes_terms = False     # `delta` may be `Combined` or `Normed`
+
+    can_norm_updates = False  # may stand on a sublayer's output (has `as_update_norm`)
+
+    def as_update_norm(self, update) -> Normed:
+        """`update` with this norm on it, for whoever adds it (a norm on a sublayer's output)."""
+        raise NotImplementedError
 
 
 class PositionEncoding(Part):

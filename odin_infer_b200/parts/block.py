@@ -14,8 +14,9 @@ class PreNormBlock(Block):
     the update it has not yet added to whoever runs next.  A block may have no feed-forward
     (and then no second norm).
 
-    post_norm_mixer / post_norm_feed_forward: a plain RMSNorm on the sublayer's output before it is added,
-    x -> x + Norm_b(Mixer(Norm(x))); the update travels as `Normed` to the norm that runs next, whose kernel sums the
+    post_norm_mixer / post_norm_feed_forward: a norm on the sublayer's output before it is added (a plain RMSNorm or a
+    layer norm), x -> x + Norm_b(Mixer(Norm(x))); with the norm "none" before the sublayer, x -> x + Norm_b(Mixer(x)).  The
+    update travels as `Normed` to the norm that runs next, whose kernel sums the
     sublayer's terms, norms them, adds and norms again.  No product then adds itself to x in its epilogue."""
 
     def __init__(self, mixer: PartSpec, feed_forward: PartSpec | None, norm_mixer: PartSpec,
@@ -27,8 +28,8 @@ class PreNormBlock(Block):
         self.post_ffn = build_part("norm", post_norm_feed_forward) if (post_norm_feed_forward is not None
                                                                         and feed_forward is not None) else None
         for post in (self.post_mixer, self.post_ffn):
-            if post is not None and (getattr(post, "groups", 1) != 1 or not hasattr(post, "weight")):
-                raise TypeError("a norm on a sublayer's output is a plain RMSNorm")
+            if post is not None and not post.can_norm_updates:
+                raise TypeError("a norm on a sublayer's output is a plain RMSNorm or a layer norm")
         self._mixer = build_part("mixer", mixer)
         self.ffn = build_part("feed_forward", feed_forward) if feed_forward is not None else None
         self.norm_mixer = build_part("norm", norm_mixer)
@@ -81,13 +82,13 @@ class PreNormBlock(Block):
         mixer, ffn = self._mixer, self.ffn
         h = self._norm(self.norm_mixer, rt, x, pending)
         if self.post_mixer is not None:
-            pending = Normed(mixer.forward(rt, step, h, entry), self.post_mixer.weight, self.post_mixer.eps)
+            pending = self.post_mixer.as_update_norm(mixer.forward(rt, step, h, entry))
         else:
             pending = mixer.forward(rt, step, h, entry, residual=x) if mixer.takes_residual else mixer.forward(rt, step, h, entry)
         if ffn is not None:
             h = self._norm(self.norm_ffn, rt, x, pending)
             if self.post_ffn is not None:
-                pending = Normed(ffn.forward(rt, step, h), self.post_ffn.weight, self.post_ffn.eps)
+                pending = self.post_ffn.as_update_norm(ffn.forward(rt, step, h))
             else:
                 pending = ffn.forward(rt, step, h, residual=x) if ffn.takes_residual else ffn.forward(rt, step, h)
         for extra in self.extras:

@@ -31,6 +31,10 @@ class RoutedExperts(FeedForward):
     score "softmax_corrected_in_groups": scores softmax(z) over all rows of the router; the experts are chosen by score +
     correction (the tensor names["router_bias"], which the weights do not see), a group's score is its largest choice
     score, and the weights are the chosen scores / (their sum + 1e-20) * route_scale.
+    score "sigmoid_as_is": the `top` largest sigmoid(z + b) are chosen and weigh with these scores * route_scale, which are
+    not divided by their sum.
+    weigh_input: a chosen expert reads its weight times h, and the update is the plain sum of the experts' answers (a shared
+    expert reads 1 * h).
     n_pass: the router has that many rows more than there are experts; a token that chooses one of them gets its own input
     back, times the weight (they count as the last members of the groups; they have no tensors).
     shared_gate: the shared expert's output is multiplied by sigmoid(g . h), one number per token, g the tensor
@@ -43,7 +47,8 @@ class RoutedExperts(FeedForward):
 
     def __init__(self, width: int, inner: int, n_experts: int, top: int, names: dict, activation: str = "silu",
                  shared_inner: int = 0, gated: bool = True, score: str = "softmax_of_chosen", groups: int = 1,
-                 keep: int = 1, route_scale: float = 1.0, shared_gate: bool = False, n_pass: int = 0):
+                 keep: int = 1, route_scale: float = 1.0, shared_gate: bool = False, n_pass: int = 0,
+                 weigh_input: bool = False):
         n_rows = n_experts + int(n_pass)
         if not (0 < top <= n_rows) or n_pass < 0:
             raise ValueError(f"every token uses {top} of {n_rows} experts: not possible")
@@ -55,12 +60,15 @@ class RoutedExperts(FeedForward):
             raise ValueError(f"a router scores by one of {', '.join(ops.ROUTER_SCORES)}, got '{score}'")
         if groups < 1 or n_rows % groups or not (1 <= keep <= groups) or keep * (n_rows // groups) < top:
             raise ValueError(f"{n_rows} experts in {groups} groups of which {keep} stay cannot give {top} experts a token")
-        if groups > 1 and score == "softmax_of_chosen":
+        if groups > 1 and score in ("softmax_of_chosen", "sigmoid_as_is"):
             raise ValueError("groups of experts go with the scores 'sigmoid_in_groups' and 'softmax_corrected_in_groups'")
         if shared_gate and not shared_inner:
             raise ValueError("a gate on the shared expert needs a shared expert")
         if shared_gate and gated:
             raise ValueError("a gate on the shared expert is built for experts without a gate matrix")
+        if weigh_input and (shared_gate or n_pass):
+            raise ValueError("weights on the experts' input go with neither a gated shared expert nor rows without an expert")
+        self.weigh_input = bool(weigh_input)
         self.width, self.inner, self.n_experts, self.top = width, inner, n_experts, top
         self.names, self.activation, self.shared_inner = dict(names), activation, int(shared_inner)
         self.gated, self.score, self.groups, self.keep = bool(gated), score, int(groups), int(keep)
@@ -146,7 +154,7 @@ class RoutedExperts(FeedForward):
         ops.moe_router(h, self.w_router, self.b_router, self.top, self.shared_as_experts, step.tok_seq, ids, wts, logits,
                        score=self.score, groups=self.groups, keep=self.keep, route_scale=self.route_scale,
                        gate_row=self.shared_gate, gate_out=gate, n_real=self.n_experts, pass_out=passed)
-        y = rt.experts(h, self.w_gate_up, self.w_down, ids, wts, self.activation, gated=self.gated)
+        y = rt.experts(h, self.w_gate_up, self.w_down, ids, wts, self.activation, gated=self.gated, weigh_input=self.weigh_input)
         if self.n_pass:
             # the input itself, times the summed weight of the chosen rows that have no expert, is one more term
             terms = Combined([ops.Term(y)])

@@ -1,4 +1,4 @@
-"""RMSNorm with a plain weight, fused with the residual add that precedes it."""
+"""Norms, fused with the residual add that precedes them: RMSNorm, layer norm, and none (the add alone)."""
 from __future__ import annotations
 
 import torch
@@ -16,6 +16,17 @@ def terms_of(update) -> list:
     if torch.is_tensor(update):
         return [ops.Term(update)]
     raise TypeError(f"an update of type {type(update).__name__} cannot be summed term by term")
+
+
+def add_terms(rt, x, delta, out, rows=None, weight=None, eps: float = 0.0, bias=None, center: bool = False) -> None:
+    """x += `delta` (None, a tensor, `Several`, `Combined`, or one of them as `Normed`), then out = norm(x), or x converted
+    without a weight (out None: the add alone); one kernel."""
+    own = delta if isinstance(delta, Normed) else None
+    update = own.update if own is not None else delta
+    terms = [] if update is None else terms_of(update)
+    ops.combine_add(x, terms, own.weight if own is not None else None, own.eps if own is not None else 0.0, weight, eps, out,
+                    rows, post_bias=own.bias if own is not None else None, post_center=own is not None and own.center,
+                    next_bias=bias, next_center=center)
 
 
 @register_part("norm", "rmsnorm")
@@ -51,6 +62,13 @@ class RMSNorm(Norm):
     def kernel_groups(self):
         return {"elementwise", "rowwise"}
 
+    def as_update_norm(self, update):
+        return Normed(update, self.weight, self.eps)
+
+    @property
+    def can_norm_updates(self) -> bool:
+        return self.groups == 1
+
     def pairs_with(self, other) -> bool:
         """Whether `other` norms the same row by the same root mean square (another weight only), so that one kernel
         can write both outputs."""
@@ -65,8 +83,7 @@ class RMSNorm(Norm):
             # a sum of terms, a norm of the update's own, the add and this norm: one kernel
             if self.groups != 1 or bias is not None or scale != 1.0 or second is not None:
                 raise TypeError("an update of several terms or with a norm of its own meets a plain RMSNorm only")
-            post_w, post_eps, inner = (delta.weight, delta.eps, delta.update) if isinstance(delta, Normed) else (None, 0.0, delta)
-            ops.combine_add(x, terms_of(inner), post_w, post_eps, self.weight, self.eps, out, rows)
+            add_terms(rt, x, delta, out, rows, self.weight, self.eps)
             return out
         if isinstance(delta, (list, tuple)) and len(delta) == 1:
             delta = delta[0]
@@ -86,3 +103,72 @@ class RMSNorm(Norm):
     def in_place(self, rt, x) -> None:
         """x (32-bit) <- its own norm."""
         ops.row_update(x, None, None, self.weight, self.eps, self.groups, x)
+
+
+@register_part("norm", "layernorm")
+class LayerNorm(Norm):
+    """o = (x - mean(x)) / sqrt(mean((x - mean(x))^2) + eps) * w + b, in 32-bit.
+
+    scale: name of a vector that multiplies the result element by element (a learned scale on a sublayer's output); it is
+    multiplied into w and b once, at load, in 32-bit."""
+
+    graph_safe = True
+    takes_several = True
+    takes_terms = True
+    can_norm_updates = True
+
+    def __init__(self, width: int, eps: float, weight: str, bias: str, scale: str | None = None):
+        self.width, self.eps, self.weight_name, self.bias_name, self.scale_name = width, float(eps), weight, bias, scale
+        self.weight = self.bias = None
+
+    def params(self):
+        out = [ParamSpec(self.weight_name, (self.width,), init="norm"), ParamSpec(self.bias_name, (self.width,), init="near_zero")]
+        if self.scale_name is not None:
+            out.append(ParamSpec(self.scale_name, (self.width,), init="unit"))
+        return out
+
+    def bind(self, tensors, rt):
+        w, b = (tensors[n].to(torch.float32) for n in (self.weight_name, self.bias_name))
+        if self.scale_name is not None:
+            s = tensors[self.scale_name].to(torch.float32)
+            w, b = w * s, b * s
+        self.weight, self.bias = w.contiguous(), b.contiguous()
+
+    def kernel_groups(self):
+        return {"rowwise"}
+
+    def as_update_norm(self, update):
+        return Normed(update, self.weight, self.eps, self.bias, True)
+
+    def forward(self, rt, x, delta, rows=None):
+        n = x.shape[0] if rows is None else rows.numel()
+        out = rt.empty(n, self.width)
+        add_terms(rt, x, Several(delta) if isinstance(delta, list) and not isinstance(delta, (Several, Combined)) else delta,
+                  out, rows, self.weight, self.eps, self.bias, True)
+        return out
+
+
+@register_part("norm", "none")
+class NoNorm(Norm):
+    """Adds what is pending to the residual stream and hands the stream on as it is, in the element type of activations (the
+    stream itself in the 32-bit engine): for sublayers that read the stream without a norm."""
+
+    graph_safe = True
+    takes_bias = True
+    takes_several = True
+    takes_terms = True
+
+    def __init__(self, width: int):
+        self.width = width
+
+    def kernel_groups(self):
+        return {"rowwise"}
+
+    def forward(self, rt, x, delta, rows=None, bias=None):
+        if rows is not None:
+            raise TypeError("this part hands on whole streams, no gathered rows")
+        if isinstance(delta, (Normed, Combined)):
+            out = None if rt.dtype == torch.float32 else rt.empty(x.shape[0], self.width)
+            add_terms(rt, x, delta, out)
+            return x if out is None else out
+        return rt.settle(x, delta, bias)

@@ -25,6 +25,7 @@ class RotaryEncoding(PositionEncoding):
     positions, lo = max(floor(p(fast)), 0), hi = min(ceil(p(slow)), rotary_dim - 1) and
     r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1), pair i turns at f_i (1 - r_i) + f_i r_i / factor, and cos and
     sin are both multiplied by 0.1 ln(factor) + 1 (the tables hold the products).
+    slowdown: every frequency is divided by it (a linear stretch of the positions).
     layout: which elements of a head form pair i: "halves" (i, i + rotary_dim / 2) or "pairs" (2i, 2i + 1); the
     tables are the same, the mixer's kernel reads the layout.
     exact_angles: position times frequency, cosine and sine are formed in double and rounded to 32-bit once (more
@@ -33,14 +34,19 @@ class RotaryEncoding(PositionEncoding):
     graph_safe = True
 
     def __init__(self, rotary_dim: int, theta: float, stretch: dict | None = None, precise: bool = False,
-                 ramp: dict | None = None, layout: str = "halves", exact_angles: bool = False):
+                 ramp: dict | None = None, layout: str = "halves", exact_angles: bool = False, slowdown: float = 1.0):
         if rotary_dim % 2:
             raise ValueError(f"rotary_dim must be even, got {rotary_dim}")
         if layout not in ("halves", "pairs"):
             raise ValueError(f"a rotation's layout is 'halves' or 'pairs', got {layout!r}")
         self.rotary_dim, self.theta, self.precise = rotary_dim, float(theta), bool(precise)
         self.layout, self.exact_angles = layout, bool(exact_angles)
+        self.slowdown = float(slowdown)
+        if not self.slowdown > 0:
+            raise ValueError(f"a rotation's slowdown must be positive, got {slowdown}")
         self.ramp, self.gain = None, 1.0
+        if self.slowdown != 1.0 and (ramp is not None or stretch is not None):
+            raise ValueError("a rotation takes one of a slowdown, a stretch by wavelength and a ramp by pair")
         if ramp is not None:
             if stretch is not None:
                 raise ValueError("a rotation takes a stretch by wavelength or a ramp by pair, not both")
@@ -59,13 +65,13 @@ class RotaryEncoding(PositionEncoding):
         """The rotary_dim / 2 frequencies as 32-bit floats."""
         half = self.rotary_dim // 2
         i = np.arange(half, dtype=np.float32)
-        if self.stretch is None and self.ramp is None and not self.precise:
+        if self.stretch is None and self.ramp is None and not self.precise and self.slowdown == 1.0:
             return (np.float32(1.0) / np.power(np.float32(self.theta), i / np.float32(max(half, 1)))).astype(np.float32)
         return self._frequencies64().astype(np.float32)
 
     def _frequencies64(self) -> np.ndarray:
         half = self.rotary_dim // 2
-        f = np.power(np.float64(self.theta), -np.arange(half, dtype=np.float64) / max(half, 1))
+        f = np.power(np.float64(self.theta), -np.arange(half, dtype=np.float64) / max(half, 1)) / self.slowdown
         if self.ramp is not None:
             rp, dims = self.ramp, self.rotary_dim
 

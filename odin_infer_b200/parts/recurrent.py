@@ -1,7 +1,7 @@
 """Mixers that keep a fixed-size state per sequence instead of keys and values.
 
-Both rest on one recurrence over a matrix-valued state S (key channel x value channel) per head,
-`ops.linear_recurrence`, held in 32-bit floats in the engine's per-sequence state area (zeroed
+All rest on a recurrence over a matrix-valued state S (key channel x value channel) per head,
+`ops.linear_recurrence` or `ops.delta_rule`, held in 32-bit floats in the engine's per-sequence state area (zeroed
 when a slot is handed out) and walked token by token; decays, gates and their exponentials are
 32-bit whatever the element type of activations.
 """
@@ -291,4 +291,80 @@ class GatedLinearAttention(Mixer):
                               q_scale=float(self.D) ** -0.5)
         y = rt.empty(T, vv)
         ops.head_unit_scale(o, self.norm_w, False, qkvg[:, 2 * qk + vv:], self.eps, y, self.H, self.V)
+        return rt.linear(y, self.w_o, out_dtype=torch.float32, may_split=True)
+
+
+@register_part("mixer", "gated_delta_rule")
+class GatedDeltaRule(Mixer):
+    """Linear attention whose write corrects what the state already answers to the token's key, with a decay.
+
+    q = W_q h, k = W_k h (n_groups x head_dim), v = W_v h (n_heads x v_head_dim), no biases; each passes a causal
+    convolution per channel (`taps` taps, the last one the current token's, no bias, zeros before the start) and SiLU.  Head
+    j reads group j // (n_heads / n_groups).  With q and k unit vectors per head (x / sqrt(sum(x^2) + unit_eps)), q also
+    times head_dim^(-1/2), beta = sigmoid(W_b h) and g = exp(-exp(A_log) softplus(W_a h + dt_bias)) per head:
+
+        S <- g S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
+
+    Each head's o goes through an RMSNorm over v_head_dim with one weight shared by the heads; the heads, side by side, are
+    multiplied by silu(W_g h) and go through W_o.  All projections of h are fused into one that leaves its sums as 32-bit;
+    the convolution's memory (its last taps - 1 inputs) and S are per-sequence state.
+    names: "q", "k", "v", "g", "b", "a", "o", "q_conv", "k_conv", "v_conv", "A_log", "dt_bias", "norm"."""
+
+    graph_safe = True
+
+    def __init__(self, width: int, n_heads: int, n_groups: int, head_dim: int, v_head_dim: int, taps: int, names: dict,
+                 eps: float = 1e-5, unit_eps: float = 1e-6):
+        if min(width, n_heads, n_groups, head_dim, v_head_dim, taps) < 1 or n_heads % n_groups:
+            raise ValueError("the delta rule needs positive sizes and heads a multiple of groups")
+        if head_dim > 256:
+            raise ValueError(f"the delta rule takes keys of up to 256 elements, got {head_dim}")
+        self.width, self.H, self.G, self.D, self.V, self.taps = width, n_heads, n_groups, head_dim, v_head_dim, taps
+        self.eps, self.unit_eps, self.names = float(eps), float(unit_eps), dict(names)
+        self.channels = 2 * n_groups * head_dim + n_heads * v_head_dim   # q | k | v, which the convolution sees
+
+    def params(self):
+        n, qk, vv = self.names, self.G * self.D, self.H * self.V
+        out = []
+        for s, rows in (("q", qk), ("k", qk), ("v", vv)):
+            out += [ParamSpec(n[s], (rows, self.width)), ParamSpec(n[s + "_conv"], (rows, self.taps), init="unit")]
+        return out + [ParamSpec(n["g"], (vv, self.width)), ParamSpec(n["b"], (self.H, self.width)),
+                      ParamSpec(n["a"], (self.H, self.width)), ParamSpec(n["A_log"], (self.H,), init="near_zero"),
+                      ParamSpec(n["dt_bias"], (self.H,), init="decay"), ParamSpec(n["norm"], (self.V,), init="norm"),
+                      ParamSpec(n["o"], (self.width, vv))]
+
+    def bind(self, tensors, rt):
+        n = self.names
+
+        def stacked(keys):
+            mats = [tensors.pop(n[s]) for s in keys]
+            if len({t.dtype for t in mats}) > 1:
+                mats = [t.float() for t in mats]
+            return torch.cat(mats, dim=0).contiguous()
+        self.w_in, self.conv_w = stacked(("q", "k", "v", "g", "b", "a")), stacked(("q_conv", "k_conv", "v_conv"))
+        self.A_log, self.dt_bias = (tensors[n[s]].to(torch.float32).contiguous() for s in ("A_log", "dt_bias"))
+        self.norm_w, self.w_o = tensors[n["norm"]], tensors[n["o"]]
+
+    def state_bytes(self) -> int:
+        return 4 * (self.H * self.D * self.V + (self.taps - 1) * self.channels)
+
+    def kernel_groups(self):
+        return {"delta_rule", "recurrent", "state_space", "gemm_plain"}
+
+    def forward(self, rt, step, h, entry):
+        T, H, qk, vv, C = h.shape[0], self.H, self.G * self.D, self.H * self.V, self.channels
+        state = _f32_view(step.state(entry))
+        n_s = H * self.D * self.V
+        S, window = state[:, :n_s], state[:, n_s:]
+        proj = rt.linear(h, self.w_in, out_dtype=torch.float32)
+        qkv = rt.empty(T, C, dtype=torch.float32)
+        ops.causal_conv(proj[:, :C], self.conv_w, None, True, window, step.tok_seq, step.seq_start, step.seq_slots,
+                        step.n_seq_cap, qkv, single_rows=step.all_single)
+        g, b, a = proj[:, C:C + vv], proj[:, C + vv:C + vv + H], proj[:, C + vv + H:]
+        o = rt.empty(T, vv, dtype=torch.float32)
+        ops.delta_rule(qkv[:, :qk], qkv[:, qk:2 * qk], qkv[:, 2 * qk:], a, b, self.A_log, self.dt_bias, o, S, step.seq_start,
+                       step.seq_slots, step.n_seq_cap, H, self.D, self.V, heads_per_group=H // self.G,
+                       q_scale=float(self.D) ** -0.5, unit_eps=self.unit_eps, block_len=_block_len(step),
+                       max_new=step.max_new)
+        y = rt.empty(T, vv)
+        ops.head_unit_scale(o, self.norm_w, False, g, self.eps, y, H, self.V)
         return rt.linear(y, self.w_o, out_dtype=torch.float32, may_split=True)

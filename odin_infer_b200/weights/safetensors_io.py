@@ -144,6 +144,7 @@ def write_safetensors(path: str, specs: Iterable[tuple[str, torch.dtype, tuple[i
                 raise SafetensorsError(f"tensor '{name}': made {t.dtype}{tuple(t.shape)}, promised {dt}{tuple(shape)}")
             t = t.contiguous().cpu()
             if t.numel():
+                t = t.reshape(-1)
                 f.write(t.view(torch.uint8).numpy().tobytes() if t.numel() < (1 << 24)
                         else memoryview(t.view(torch.uint8).numpy()))
     os.replace(tmp, path)

@@ -46,7 +46,7 @@ def read_model_folder(folder: str, dtype=torch.float32):
             raw = np.frombuffer(f.read(e - b), dtype=npdt).reshape(meta["shape"])
             if meta["dtype"] == "BF16":
                 # a bfloat16 is the upper half of a float32
-                t = torch.from_numpy((raw.astype(np.uint32) << 16).view(np.float32).copy())
+                t = torch.from_numpy(np.asarray(raw.astype(np.uint32) << 16, dtype=np.uint32).view(np.float32).copy())
             else:
                 t = torch.from_numpy(raw.copy())
             tensors[name] = t.to(dtype) if t.is_floating_point() else t
