@@ -1144,6 +1144,231 @@ def meropel_workload(steps: int, warmup: int) -> int:
     return 0
 
 
+# --------------------------------------------------------------------------------------------------------------
+# --workload fugavik: the Fugavik design beside the Nikonex design (the closest: latent attention, a matrix-state recurrence,
+# experts chosen by sigmoid scores)
+# --------------------------------------------------------------------------------------------------------------
+FUGAVIK_SIZES = {
+    # the Nikonex sizes' width, layers, vocabulary and experts, its retention's heads for the delta rule (keys and queries of
+    # half as many heads) and its latent row's size; attention of 16 (32) query heads on 8 kv heads of 128; dense
+    # feed-forwards of three times the width
+    "2048": dict(NIKONEX_SIZES["2048"], delta_heads=16, delta_kv=8, delta_dim=128, delta_v=128, latent_row=128, dense=6144),
+    "4096": dict(NIKONEX_SIZES["4096"], delta_heads=32, delta_kv=16, delta_dim=128, delta_v=128, latent_row=128, dense=12288),
+}
+
+
+def fugavik_config(z: dict) -> dict:
+    att = {"heads": z["heads"], "kv_heads": z["kv"], "dim": z["hd"], "vdim": z["hd"], "scale": z["hd"] ** -0.5, "v_mix": True,
+           "rot": {"dims": z["hd"], "base": 500000.0, "scaling": {"factor": 4.0}}}
+    lat = {"heads": z["lat_heads"], "dim": z["lat_dim"], "vdim": z["lat_v"], "kv_rank": z["latent_row"], "scale": z["lat_dim"] ** -0.5}
+    dlt = {"heads": z["delta_heads"], "kv_heads": z["delta_kv"], "dim": z["delta_dim"], "vdim": z["delta_v"], "conv": 4}
+    moe = {"kind": "moe", "expert": {"ff": z["eff"]}, "router": {"experts": z["experts"], "top": z["top"]}}
+    dense = {"kind": "dense", "ff": z["dense"]}
+    cycle = [("delta", dlt, moe), ("attention", att, dense), ("latent_attention", lat, moe), ("attention", att, dense)]
+    layers = [{"type": t, "mixer": m, "mlp": f} for t, m, f in (cycle[i % 4] for i in range(z["layers"]))]
+    return {"architecture": "Fugavik", "vocab": z["vocab"], "width": z["width"], "norm": {"eps": 1e-5}, "layers": layers}
+
+
+def fugavik_kernels(z: dict, T: int, peaks: dict) -> dict:
+    """Every kernel that the design adds (or runs with options of its own), alone at this size for T token rows (one
+    prompt of T tokens, or T sequences of one token after 512), beside the like kernel of the closest existing path:
+    microseconds, and algorithmic bytes (or FLOPs) over the time as a fraction of the measured peaks."""
+    import torch
+    from odin_infer_b200.csrc import ops
+    from odin_infer_b200.engine import runtime as R
+    dev, bf = "cuda:0", torch.bfloat16
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    d, E, top, eff, ff = z["width"], z["experts"], z["top"], z["eff"], z["dense"]
+    decode = T <= 64
+    out = {}
+
+    def replayed(fn, flush, reps=5, inner=20):
+        fn()
+        torch.cuda.synchronize()
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            for _ in range(inner):
+                fn()
+        return _timed(graph.replay, flush, reps) / inner
+    timed = replayed if decode else _timed
+
+    def note(name, us, nbytes=None, flops=None, **more):
+        rec = {"us": round(us, 2)}
+        if nbytes is not None:
+            rec["of_hbm"] = round(nbytes / (us * 1e-6) / 1e9 / peaks["hbm_gbs"], 3)
+        if flops is not None:
+            rec["tflops"] = round(flops / (us * 1e-6) / 1e12, 2)
+        rec.update(more)
+        out[name] = rec
+    rt = R.Runtime(dev, bf)
+    torch.manual_seed(0)
+    ctx = 512 if decode else 0
+    n_seq = T if decode else 1
+    per_seq = (ctx + 1 + 63) // 64 if decode else (T + 63) // 64
+    n_pages = n_seq * per_seq
+    bt = torch.arange(n_pages, dtype=torch.int32, device=dev).reshape(n_seq, per_seq).contiguous()
+    pos = torch.full((T,), ctx, dtype=torch.int32, device=dev) if decode else torch.arange(T, dtype=torch.int32, device=dev)
+    seq = torch.arange(T, dtype=torch.int32, device=dev) if decode else torch.zeros(T, dtype=torch.int32, device=dev)
+    starts = torch.arange(0, T + 1, 1 if decode else T, dtype=torch.int32, device=dev)
+    slots = torch.arange(n_seq, dtype=torch.int32, device=dev)
+    h = torch.randn(T, d, device=dev).to(bf)
+    x = torch.randn(T, d, device=dev)
+    w1, b1 = torch.randn(d, device=dev), torch.randn(d, device=dev)
+    hb = torch.empty(T, d, dtype=bf, device=dev)
+    # the residual stream: the update's layer norm with its scale, the add, the stream converted for the next sublayer
+    d1 = torch.randn(T, d, device=dev)
+    nb = T * d * (4 * 3 + 2)
+    note("add + RMSNorm of an update (nikonex)", timed(lambda: ops.row_update(x, [d1, d1], None, w1, 1e-6, 1, hb, scale=0.6), flush), nbytes=nb + T * d * 4)
+    note("an update's RMSNorm, the add, the next norm (meropel)", timed(
+        lambda: ops.combine_add(x, [ops.Term(d1)], w1, 1e-6, w1, 1e-6, hb), flush), nbytes=nb)
+    note("an update's layer norm with a bias, the add, the stream in bfloat16", timed(
+        lambda: ops.combine_add(x, [ops.Term(d1)], w1, 1e-5, None, 0.0, hb, post_bias=b1, post_center=True), flush), nbytes=nb)
+    # head preparation with values mixed, beside the one without
+    Hq, Hkv, hd = z["heads"], z["kv"], z["hd"]
+    kc = (torch.randn(n_pages, Hkv, 64, hd, device=dev) * 0.3).to(bf)
+    vc = (torch.randn(n_pages, Hkv, 64, hd, device=dev) * 0.3).to(bf)
+    qkv = torch.randn(T, (Hq + 2 * Hkv) * hd, device=dev).to(bf)
+    hn = torch.ones(hd, dtype=bf, device=dev)
+    ch = torch.randn(max(T, ctx + 1), hd // 2, device=dev)
+    q_out = torch.empty(T, Hq * hd, dtype=bf, device=dev)
+    v1 = torch.randn(T, Hkv * hd, device=dev).to(bf)
+    pb = T * (Hq + 2 * Hkv) * hd * 4
+    note("head preparation (nikonex's neighbour nufupel)", timed(
+        lambda: ops.head_prep(qkv, Hq, Hkv, hd, hn, hn, 1e-6, ch, ch, hd, pos, seq, bt, kc, vc, q_out=q_out), flush), nbytes=pb)
+    note("head preparation, values kept for later layers", timed(
+        lambda: ops.head_prep(qkv, Hq, Hkv, hd, hn, hn, 1e-6, ch, ch, hd, pos, seq, bt, kc, vc, q_out=q_out, v_keep=v1), flush), nbytes=pb + T * Hkv * hd * 2)
+    note("head preparation, values mixed with the first layer's", timed(
+        lambda: ops.head_prep(qkv, Hq, Hkv, hd, hn, hn, 1e-6, ch, ch, hd, pos, seq, bt, kc, vc, q_out=q_out, v_first=v1, v_lambda=0.4), flush), nbytes=pb + T * Hkv * hd * 2)
+    # attention with a sink over keys and values of the cache, and over latent rows
+    H, e, ev, L = z["lat_heads"], z["lat_dim"], z["lat_v"], z["latent_row"]
+    rows = (torch.randn(n_pages, 1, 64, L, device=dev) * 0.3).to(bf)
+    qf, of = torch.randn(T, H * L, device=dev).to(bf), torch.empty(T, H * L, dtype=bf, device=dev)
+    sinks = {n: torch.randn(n, device=dev) for n in (Hq, H)}
+    for name, qq, nq, nkv, dim, k_, v_ in (("", q_out, Hq, Hkv, hd, kc, vc), (" over shared rows", qf, H, 1, L, rows, rows)):
+        for sk, tag in ((None, " (nikonex)"), (sinks[nq], ", a sink")):
+            oo = torch.empty_like(qq)
+            if decode:
+                n_split = R.decode_key_splits(T, nkv, ctx + 1)
+                scratch = torch.empty(ops.attention_decode_scratch(T, nq, dim, n_split), dtype=torch.float32, device=dev)
+                note("decode attention over 512 keys" + name + tag, timed(
+                    lambda: ops.attention_decode(qq, oo, nq, nkv, dim, k_, v_, pos, seq, bt, 0, scratch, n_split, 0, dim ** -0.5, 0.0, sk), flush),
+                    nbytes=T * (ctx + 1) * nkv * dim * 2 * (2 if k_ is not v_ else 1))
+            else:
+                lens = torch.tensor([T], dtype=torch.int32, device=dev)
+                note("prompt attention" + name + tag, timed(
+                    lambda: ops.attention_prefill(qq, oo, 1, T, nq, nkv, dim, k_, v_, starts, lens, bt, 0, 0, dim ** -0.5, 0.0, sk), flush),
+                    flops=4.0 * nq * dim * T * (T + 1) / 2)
+    # around latent attention: the cached row, the products per head without and with the gate
+    down = torch.randn(T, H * e + L + H, device=dev).to(bf)
+    cn, dummy = torch.ones(L, dtype=bf, device=dev), torch.zeros(1, 1, device=dev)
+    note("latent preparation (norm, cache row)", timed(
+        lambda: ops.latent_prep(down[:, H * e:H * e + L], 0, L, 0, False, None, cn, 1e-5, None, dummy, dummy, pos, seq, bt, rows), flush), nbytes=T * L * 4)
+    w_uk = (torch.randn(H, e, L, device=dev) / e ** 0.5).to(bf)
+    w_uv = (torch.randn(H, L, ev, device=dev) / L ** 0.5).to(bf)
+    ov = torch.empty(T, H * ev, dtype=bf, device=dev)
+    note("queries onto the latent, a product per head (nikonex)", timed(lambda: ops.heads_linear(down, e, w_uk, qf, L), flush),
+         flops=2.0 * T * H * e * L, nbytes=T * H * (e + L) * 2 + w_uk.numel() * 2)
+    note("values from the latent, a product per head (nikonex)", timed(lambda: ops.heads_linear(of, L, w_uv, ov, ev), flush),
+         flops=2.0 * T * H * L * ev, nbytes=T * H * (L + ev) * 2 + w_uv.numel() * 2)
+    note("values from the latent, a product per head, times the head's gate", timed(
+        lambda: ops.heads_linear(of, L, w_uv, ov, ev, gate=down[:, H * e + L:]), flush),
+        flops=2.0 * T * H * L * ev, nbytes=T * H * (L + ev) * 2 + w_uv.numel() * 2)
+    # the delta rule beside retention's recurrence at equal heads and sizes, with its convolution and the heads' norm
+    RH, G, dk, dv = z["delta_heads"], z["delta_kv"], z["delta_dim"], z["delta_v"]
+    blocks = dict(block_len=128, max_new=T) if not decode else {}
+    tag = " in blocks of 128 tokens" if not decode else ""
+    C = 2 * G * dk + RH * dv
+    proj, act = torch.randn(T, C + RH * dv + 2 * RH, device=dev), torch.empty(T, C, device=dev)
+    cw, cstate = torch.randn(C, 4, device=dev).to(bf), torch.zeros(n_seq, 3 * C, device=dev)
+    note(f"causal convolution of 4 taps over {C} channels with SiLU, and its memory", timed(
+        lambda: ops.causal_conv(proj[:, :C], cw, None, True, cstate, seq, starts, slots, n_seq, act, single_rows=decode), flush),
+        nbytes=T * C * 8 + 2 * n_seq * 3 * C * 4)
+    state = torch.zeros(n_seq, RH * dk * dv, device=dev)
+    rb = 4 * (T * (2 * RH * dk + 2 * RH * dv) + 2 * n_seq * RH * dk * dv)
+    db = 4 * (T * (2 * G * dk + 2 * RH * dv + 2 * RH) + 2 * n_seq * RH * dk * dv)
+    q, k, v, ro = (torch.randn(T, RH * n, device=dev) for n in (dk, dk, dv, dv))
+    decay, sb = torch.full((RH,), 0.99, device=dev), torch.randn(RH, device=dev) - 2
+    note(f"recurrence with a fixed decay ({RH} heads of {dk} x {dv}; nikonex)" + tag, timed(
+        lambda: ops.linear_recurrence("fixed", q, k, None, v, decay, decay, ro, state, starts, slots, n_seq, RH, dk, dv, **blocks), flush),
+        nbytes=rb, flops=T * RH * 4.0 * dk * dv)
+    state.zero_()
+    note(f"delta rule ({RH} heads of {dk} x {dv}, {G} of q and k)" + (" in chunks of 64 tokens" if not decode else ""), timed(
+        lambda: ops.delta_rule(act[:, :G * dk], act[:, G * dk:2 * G * dk], act[:, 2 * G * dk:], proj[:, C + RH * dv:C + RH * dv + RH],
+                               proj[:, C + RH * dv + RH:], sb * 0, sb, ro, state, starts, slots, n_seq, RH, dk, dv,
+                               heads_per_group=RH // G, q_scale=dk ** -0.5, chunked=not decode, max_new=T), flush), nbytes=db, flops=T * RH * 8.0 * dk * dv)
+    y, wn = torch.empty(T, RH * dv, dtype=bf, device=dev), torch.ones(dv, dtype=bf, device=dev)
+    note("heads' unit norm times silu(gate) (nikonex)", timed(lambda: ops.head_unit_scale(ro, None, False, proj[:, C:C + RH * dv], 1e-5, y, RH, dv), flush), nbytes=T * RH * dv * 10)
+    note("heads' norm with a shared weight times silu(gate)", timed(lambda: ops.head_unit_scale(ro, wn, False, proj[:, C:C + RH * dv], 1e-5, y, RH, dv), flush), nbytes=T * RH * dv * 10)
+    # router and experts: weights on what the experts read, beside weights on what they answer; the dense feed-forward
+    wr = (torch.randn(E, d, device=dev) / d ** 0.5).to(bf)
+    ids = torch.empty(T, top, dtype=torch.int32, device=dev)
+    wts = torch.empty(T, top, dtype=torch.float32, device=dev)
+
+    def route(score, **kw):
+        lg = rt.linear(h, wr, out_dtype=torch.float32) if T > 64 else None
+        ops.moe_router(h, wr, None, top, 0, seq, ids, wts, lg, score=score, **kw)
+    rb = T * d * 2 + E * d * 2
+    note("router, sigmoid scores in groups (nikonex)", timed(lambda: route("sigmoid_in_groups", groups=z["groups"], keep=z["keep"]), flush), nbytes=rb)
+    note("router, sigmoid scores as they are", timed(lambda: route("sigmoid_as_is"), flush), nbytes=rb)
+    used = len(torch.unique(ids))
+    wg = (torch.randn(E, 2 * eff, d, device=dev) * 0.02).to(bf)
+    wd = (torch.randn(E, d, eff, device=dev) * 0.02).to(bf)
+    for name, kw in (("weights on their answers (nufupel)", {}), ("weights on their inputs", dict(weigh_input=True))):
+        note(f"experts with a gate matrix, {name}; all their launches", timed(lambda: rt.experts(h, wg, wd, ids, wts, "silu", **kw), flush),
+             flops=2.0 * T * top * 3 * eff * d, nbytes=used * 3 * eff * d * 2, experts_used=used)
+    wgu, wup, wdn = ((torch.randn(n, m, device=dev) * 0.02).to(bf) for n, m in ((2 * ff, d), (ff, d), (d, ff)))
+
+    def dense(kind):
+        if kind == "swiglu":
+            a = rt.gated_linear(h, wgu, ff)
+        else:
+            a = rt.activated_linear(h, wup, "relu2")
+        return rt.linear(a, wdn, out_dtype=torch.float32, may_split=True)
+    note("dense feed-forward with SwiGLU (nufupel)", timed(lambda: dense("swiglu"), flush), flops=2.0 * T * 3 * d * ff, nbytes=3 * d * ff * 2)
+    note("dense feed-forward with relu squared", timed(lambda: dense("relu2"), flush), flops=2.0 * T * 2 * d * ff, nbytes=2 * d * ff * 2)
+    torch.cuda.synchronize()
+    return out
+
+
+def fugavik_workload(steps: int, warmup: int) -> int:
+    """The Fugavik design at two sizes that resemble a real model's layers, beside the Nikonex design of the same
+    width, layers, vocabulary and experts (random weights): a prompt of 2,048 tokens in one step, decoding at batch 8
+    after 512-token prompts (device-timed), and every kernel of the design alone beside its like."""
+    import torch
+    from odin_infer_b200 import Engine, Engine_Opts
+    from odin_infer_b200.config import config_from_dict
+    from odin_infer_b200.csrc import ops
+    peaks, peak_source = load_peaks()
+    result = {"metric": "Fugavik beside Nikonex at equal sizes: prompt of 2,048 tokens, decode at batch 8 (512-token prompts), "
+                        "bf16, random weights", "peak_source": peak_source, "sizes": {}}
+    steps = min(steps, 64)
+    for name, z in FUGAVIK_SIZES.items():
+        entry = {}
+        for model, raw in (("fugavik", fugavik_config(z)), ("nikonex", nikonex_config(z))):
+            need = PROMPT + warmup + steps + 72
+            engine = Engine.random(config_from_dict(raw), WEIGHT_SEED, Engine_Opts(
+                max_ctx=CONTEXT, max_tokens=max(8 * ((need + 63) // 64 * 64), PREFILL_TOKENS + 64), max_batch=8,
+                dtype="bfloat16", verbose=False))
+            ms_pf = run_prefill(engine, z["vocab"])
+            tps, ms_step, _, launches = run_decode(engine, 8, steps, warmup, z["vocab"])
+            entry[model] = {"layers": z["layers"], "weights_gib": round(engine.weight_bytes / 2 ** 30, 2),
+                            "prefill_2048": {"ms": round(ms_pf, 3), "tokens_per_s": round(PREFILL_TOKENS / ms_pf * 1e3)},
+                            "decode_b8": {"ms_per_step": round(ms_step, 4), "tokens_per_s": round(tps, 1),
+                                          "launches_per_step": launches // steps}}
+            engine.destroy()
+            del engine
+            torch.cuda.empty_cache()
+        entry["kernels_prompt_2048_rows"] = fugavik_kernels(z, PREFILL_TOKENS, peaks)
+        entry["kernels_decode_8_rows"] = fugavik_kernels(z, 8, peaks)
+        result["sizes"][name] = entry
+    ops.gemm_tc_check()
+    ops.attention_prefill_check()
+    ops.attention_decode_check()
+    ops.moe_tc_check()
+    print(json.dumps(result))
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1155,13 +1380,14 @@ def main() -> int:
     ap.add_argument("--no-points", action="store_true", help="skip the batch 1 / 64 points and the prefill")
     ap.add_argument("--no-graphs", action="store_true", help="launch the decode step's kernels one by one (for profilers)")
     ap.add_argument("--no-e2e", action="store_true", help="skip the end-to-end run (for profilers)")
-    ap.add_argument("--workload", default="8b", choices=["8b", "1.7b-mixed", "32b-long", "tovalix", "nufupel", "nikonex", "meropel"],
+    ap.add_argument("--workload", default="8b", choices=["8b", "1.7b-mixed", "32b-long", "tovalix", "nufupel", "nikonex", "meropel", "fugavik"],
                     help="8b: the contract's run (default).  The others are further workloads of the baseline's list and "
                          "print a line of their own: 1.7b-mixed = Qwen3-1.7B shape, 64 prompts of 16..2048 tokens, 128 new "
                          "tokens each; 32b-long = Qwen3-32B shape, a 2,048-token prompt, decoding 1 and 8 sequences at context 8192; "
                          "tovalix = the Tovalix design beside the Qwen3 decoder at equal sizes, and its kernels alone; "
                          "nufupel = the same for the Nufupel design; nikonex = the Nikonex design beside Nufupel at equal sizes, "
-                         "and its kernels alone; meropel = the Meropel design beside Nikonex at equal sizes, and its kernels alone")
+                         "and its kernels alone; meropel, fugavik = the Meropel or the Fugavik design beside Nikonex at equal sizes, and its "
+                         "kernels alone")
     args = ap.parse_args()
 
     if args.impl == "reference":
@@ -1181,6 +1407,8 @@ def main() -> int:
         return nikonex_workload(args.steps, warmup)
     if args.workload == "meropel":
         return meropel_workload(args.steps, warmup)
+    if args.workload == "fugavik":
+        return fugavik_workload(args.steps, warmup)
     if args.workload != "8b":
         return other_workload(args.workload)
 

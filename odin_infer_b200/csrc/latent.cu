@@ -110,6 +110,7 @@ extern "C" int odin_latent_prep(const void* down, int in_dtype, int n_split, lon
 // a number per token and head, itself possibly partial sums; the sum is multiplied by its sigmoid.
 #define HL_THREADS 128
 #define HL_TOK 8
+#define HL_PRE 32
 
 struct HeadGate {
     const void* p;             // null: no gate
@@ -141,40 +142,65 @@ heads_linear_kernel(const TA* __restrict__ a, int a_splits, size_t a_ss, size_t 
     pdl_trigger();
     const int h = blockIdx.y, t0 = blockIdx.z * HL_TOK;
     const int n = blockIdx.x * HL_THREADS + threadIdx.x;
+    // a column's weights come HL_PRE at a time, the first ones while the kernel before this one still runs, the next ones
+    // while the ones before them are multiplied: with few tokens the kernel is a chain of trips to memory otherwise
+    const TW* wh = w + (size_t)h * K * N + n;
+    TW cur[HL_PRE], nxt[HL_PRE];
+    auto fetch = [&](TW (&dst)[HL_PRE], int k0) {
+#pragma unroll
+        for (int j = 0; j < HL_PRE; ++j)
+            if (n < N && k0 + j < K) dst[j] = wh[(size_t)(k0 + j) * N];
+    };
+    fetch(cur, 0);
     pdl_wait();
-    for (int e = threadIdx.x; e < K * HL_TOK; e += blockDim.x) {
-        const int u = e / K, k = e % K;
-        as[k * HL_TOK + u] = (t0 + u < T) ? sum_parts(a, (size_t)(t0 + u) * a_rs + (size_t)h * a_hs + k, a_splits, a_ss) : 0.f;
+    {   // sixteen threads per token; a thread's loads of one part go out together
+        const int u = threadIdx.x / (HL_THREADS / HL_TOK), l = threadIdx.x % (HL_THREADS / HL_TOK);
+        const TA* ar = a + (size_t)(t0 + u) * a_rs + (size_t)h * a_hs;
+        for (int k0 = l; k0 < K; k0 += 8 * (HL_THREADS / HL_TOK)) {
+            float v[8];
+#pragma unroll
+            for (int j = 0; j < 8; ++j) v[j] = 0.f;
+            for (int sp = 0; sp < a_splits; ++sp) {
+#pragma unroll
+                for (int j = 0; j < 8; ++j) {
+                    const int k = k0 + j * (HL_THREADS / HL_TOK);
+                    if (k < K && t0 + u < T) v[j] += to_f32(ar[(size_t)sp * a_ss + k]);
+                }
+            }
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                const int k = k0 + j * (HL_THREADS / HL_TOK);
+                if (k < K) as[k * HL_TOK + u] = v[j];
+            }
+        }
     }
+    __shared__ float factors[HL_TOK];
+    if (threadIdx.x < HL_TOK) factors[threadIdx.x] = t0 + threadIdx.x < T ? gate.factor(t0 + threadIdx.x, h) : 1.0f;
     __syncthreads();
     if (n >= N) return;
-    const TW* wh = w + (size_t)h * K * N + n;
     float acc[HL_TOK];
 #pragma unroll
     for (int u = 0; u < HL_TOK; ++u) acc[u] = 0.f;
-    int k = 0;
-    for (; k + 4 <= K; k += 4) {
-        float wv[4];
+    for (int k0 = 0; k0 < K; k0 += HL_PRE) {
+        fetch(nxt, k0 + HL_PRE);
 #pragma unroll
-        for (int j = 0; j < 4; ++j) wv[j] = to_f32(wh[(size_t)(k + j) * N]);
-#pragma unroll
-        for (int j = 0; j < 4; ++j) {
-            const float4 a0 = *reinterpret_cast<const float4*>(&as[(k + j) * HL_TOK]);
-            const float4 a1 = *reinterpret_cast<const float4*>(&as[(k + j) * HL_TOK + 4]);
-            acc[0] = fmaf(wv[j], a0.x, acc[0]); acc[1] = fmaf(wv[j], a0.y, acc[1]);
-            acc[2] = fmaf(wv[j], a0.z, acc[2]); acc[3] = fmaf(wv[j], a0.w, acc[3]);
-            acc[4] = fmaf(wv[j], a1.x, acc[4]); acc[5] = fmaf(wv[j], a1.y, acc[5]);
-            acc[6] = fmaf(wv[j], a1.z, acc[6]); acc[7] = fmaf(wv[j], a1.w, acc[7]);
+        for (int j = 0; j < HL_PRE; ++j) {
+            if (k0 + j < K) {
+                const float wv = to_f32(cur[j]);
+                const float4 a0 = *reinterpret_cast<const float4*>(&as[(k0 + j) * HL_TOK]);
+                const float4 a1 = *reinterpret_cast<const float4*>(&as[(k0 + j) * HL_TOK + 4]);
+                acc[0] = fmaf(wv, a0.x, acc[0]); acc[1] = fmaf(wv, a0.y, acc[1]);
+                acc[2] = fmaf(wv, a0.z, acc[2]); acc[3] = fmaf(wv, a0.w, acc[3]);
+                acc[4] = fmaf(wv, a1.x, acc[4]); acc[5] = fmaf(wv, a1.y, acc[5]);
+                acc[6] = fmaf(wv, a1.z, acc[6]); acc[7] = fmaf(wv, a1.w, acc[7]);
+            }
         }
-    }
-    for (; k < K; ++k) {
-        const float wv = to_f32(wh[(size_t)k * N]);
 #pragma unroll
-        for (int u = 0; u < HL_TOK; ++u) acc[u] = fmaf(wv, as[k * HL_TOK + u], acc[u]);
+        for (int j = 0; j < HL_PRE; ++j) cur[j] = nxt[j];
     }
 #pragma unroll
     for (int u = 0; u < HL_TOK; ++u)
-        if (t0 + u < T) out[(size_t)(t0 + u) * o_rs + (size_t)h * o_hs + n] = from_f32<TO>(acc[u] * gate.factor(t0 + u, h));
+        if (t0 + u < T) out[(size_t)(t0 + u) * o_rs + (size_t)h * o_hs + n] = from_f32<TO>(acc[u] * factors[u]);
 }
 
 // Many tokens: a CTA takes 64 tokens by 64 output channels of one head, K in steps of 32 through shared memory, a thread

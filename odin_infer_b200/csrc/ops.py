@@ -606,10 +606,13 @@ def linear_recurrence(mode: str, q: torch.Tensor, k: torch.Tensor | None, g: tor
         "linear_recurrence", kernels=kernels)
 
 
+DELTA_CHUNK = 64   # tokens of a chunk of the delta rule's form for long prompts
+
+
 def delta_rule(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a: torch.Tensor, b: torch.Tensor, A_log: torch.Tensor,
                a_bias: torch.Tensor, out: torch.Tensor, state: torch.Tensor, seq_start: torch.Tensor,
                seq_slots: torch.Tensor, n_seqs: int, n_heads: int, dk: int, dv: int, heads_per_group: int = 1,
-               q_scale: float = 1.0, unit_eps: float = 1e-6, block_len: int = 0, max_new: int = 0) -> None:
+               q_scale: float = 1.0, unit_eps: float = 1e-6, chunked: bool = False, max_new: int = 0) -> None:
     """The gated delta rule over a state S [dk, dv] per (sequence, head) in `state` (float32 [slots, >= H dk dv], any row
     stride), sequence t's rows in order.  With u(x) = x / sqrt(sum(x^2) + unit_eps) over a head's dk elements,
     g = exp(-exp(A_log[h]) softplus(a[t, h] + a_bias[h])) and beta = sigmoid(b[t, h]):
@@ -619,31 +622,30 @@ def delta_rule(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a: torch.Tenso
     q, k: float32 [T, (H / heads_per_group) dk] (head h reads group h // heads_per_group), v, out: float32 [T, H dv],
     a, b: float32 [T, H]; all may be strided views.  A_log, a_bias: [H] of one element type.
 
-    block_len > 0 (with max_new, the most rows any sequence brings): every sequence's rows are cut into blocks of
-    block_len tokens that are walked side by side, each from zeros and with its transition matrix; two kernels then carry
-    the state from block to block and add each block's incoming state to its tokens' outputs.  The same values up to
-    rounding; for long prompts."""
+    chunked (with max_new, the most rows any sequence brings): for long prompts.  Every sequence's rows are cut into chunks
+    of DELTA_CHUNK tokens; one kernel solves each chunk's writes as functions of the state at its start, a second carries
+    the state from chunk to chunk, a third forms the outputs.  The same values up to rounding."""
     T = q.shape[0]
     for t, n in ((q, n_heads // heads_per_group * dk), (k, n_heads // heads_per_group * dk), (v, n_heads * dv),
                  (out, n_heads * dv), (a, n_heads), (b, n_heads)):
         assert t.dtype == torch.float32 and (t.stride(1) == 1 or n == 1) and tuple(t.shape) == (T, n)
     assert state.dtype == torch.float32 and state.stride(1) == 1 and state.shape[1] >= n_heads * dk * dv
     assert A_log.numel() == a_bias.numel() == n_heads and A_log.dtype == a_bias.dtype
-    n_blocks, qp, s_loc, m_loc, kernels = 0, None, None, None, 1
-    if block_len > 0:
+    n_chunks, scratch = 0, None
+    if chunked:
         assert max_new > 0
-        n_blocks = (max_new + block_len - 1) // block_len
-        qp = torch.empty(T, n_heads * dk, dtype=torch.float32, device=q.device)
-        s_loc = torch.empty(n_seqs * n_blocks, n_heads * dk * dv, dtype=torch.float32, device=q.device)
-        m_loc = torch.empty(n_seqs * n_blocks, n_heads * dk * dk, dtype=torch.float32, device=q.device)
-        kernels = 3
+        n_chunks = (max_new + DELTA_CHUNK - 1) // DELTA_CHUNK
+        f = build.load("delta_rule").odin_delta_rule_scratch
+        f.restype = c_longlong
+        floats = int(f(c_int(T), c_int(n_seqs), c_int(n_heads), c_int(dk), c_int(dv)))
+        scratch = torch.empty(floats, dtype=torch.float32, device=q.device)
     _check(_fn("delta_rule", "odin_delta_rule")(
         _ptr(q), c_longlong(q.stride(0)), _ptr(k), c_longlong(k.stride(0)), _ptr(v), c_longlong(v.stride(0)),
         _ptr(a), c_longlong(a.stride(0)), _ptr(b), c_longlong(b.stride(0)), _ptr(A_log), _ptr(a_bias),
         c_int(dtype_code(A_log.dtype)), _ptr(out), c_longlong(out.stride(0)), _ptr(state), c_longlong(state.stride(0)),
         _ptr(seq_start), _ptr(seq_slots), c_int(n_seqs), c_int(n_heads), c_int(dk), c_int(dv), c_int(heads_per_group),
-        c_float(q_scale), c_float(unit_eps), c_int(block_len), c_int(n_blocks), _ptr(qp), _ptr(s_loc), _ptr(m_loc),
-        _stream()), "delta_rule", kernels=kernels)
+        c_float(q_scale), c_float(unit_eps), c_int(T), c_int(n_chunks), _ptr(scratch), _stream()), "delta_rule",
+        kernels=3 if chunked else 1)
 
 
 def causal_conv(src: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | None, silu: bool, state: torch.Tensor,

@@ -223,6 +223,13 @@ class Runtime:
         ops.swiglu(self.linear(a, w_gate_up, may_split=True), act)
         return act
 
+    def activated_linear(self, a: torch.Tensor, w: torch.Tensor, activation: str, params: torch.Tensor | None = None) -> torch.Tensor:
+        """act(a W^T): a product followed by the activation kernel (which also adds the partial sums of a split product).
+        activation: one of `ops.ACTIVATIONS`; params: its numbers, where it has any."""
+        act = self.empty(a.shape[0], w.shape[0])
+        ops.activation(self.linear(a, w, may_split=True), activation, act, params)
+        return act
+
     # ---- experts chosen per token ----------------------------------------
     def experts(self, h: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor,
                 wts: torch.Tensor, activation: str, gated: bool = True, weigh_input: bool = False) -> torch.Tensor:

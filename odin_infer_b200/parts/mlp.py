@@ -83,7 +83,5 @@ class ActivatedMLP(FeedForward):
         return {"rowwise", "gemm_plain"}
 
     def forward(self, rt, step, h, residual=None):
-        up = rt.linear(h, self.w_up, may_split=True)
-        act = rt.empty(h.shape[0], self.inner)
-        ops.activation(up, self.activation, act, self.act_params)
+        act = rt.activated_linear(h, self.w_up, self.activation, self.act_params)
         return rt.linear(act, self.w_down, out_dtype=torch.float32, may_split=True, add_to=residual)

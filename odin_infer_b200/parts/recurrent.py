@@ -19,6 +19,10 @@ RECURRENCE_BLOCK = 128
 BLOCKS_FROM = 2 * RECURRENCE_BLOCK
 
 
+# A step in which a sequence brings this many tokens or more runs the delta rule chunk by chunk (see ops.delta_rule).
+DELTA_CHUNKS_FROM = 2 * ops.DELTA_CHUNK
+
+
 def _block_len(step) -> int:
     return RECURRENCE_BLOCK if step.max_new >= BLOCKS_FROM else 0
 
@@ -363,8 +367,8 @@ class GatedDeltaRule(Mixer):
         o = rt.empty(T, vv, dtype=torch.float32)
         ops.delta_rule(qkv[:, :qk], qkv[:, qk:2 * qk], qkv[:, 2 * qk:], a, b, self.A_log, self.dt_bias, o, S, step.seq_start,
                        step.seq_slots, step.n_seq_cap, H, self.D, self.V, heads_per_group=H // self.G,
-                       q_scale=float(self.D) ** -0.5, unit_eps=self.unit_eps, block_len=_block_len(step),
-                       max_new=step.max_new)
+                       q_scale=float(self.D) ** -0.5, unit_eps=self.unit_eps,
+                       chunked=step.max_new >= DELTA_CHUNKS_FROM, max_new=step.max_new)
         y = rt.empty(T, vv)
         ops.head_unit_scale(o, self.norm_w, False, g, self.eps, y, H, self.V)
         return rt.linear(y, self.w_o, out_dtype=torch.float32, may_split=True)
