@@ -167,16 +167,29 @@ def relu2_mlp(x, up, down, rnd=_same):
     return rnd(torch.relu(x @ up.T) ** 2) @ down.T
 
 
-def route(x, w_router, router: dict):
-    """Per token the chosen (expert, weight) pairs, best first."""
-    s = torch.sigmoid(x @ w_router.T)
-    return [[(e, float(row[e])) for e in sorted(range(router["experts"]), key=lambda e: (-float(row[e]), e))[:router["top"]]]
-            for row in s]
+def route(x, w_router, router: dict, swapped=()):
+    """Per token the chosen (expert, weight) pairs, best first.  swapped: tokens for which the last choice and the best
+    expert that is not chosen change places (a close call taken the other way)."""
+    s, top, out = torch.sigmoid(x @ w_router.T), router["top"], []
+    for t, row in enumerate(s):
+        order = sorted(range(router["experts"]), key=lambda e: (-float(row[e]), e))
+        if t in swapped:
+            order[top - 1], order[top] = order[top], order[top - 1]
+        out.append([(e, float(row[e])) for e in order[:top]])
+    return out
 
 
-def expert_mlp(x, w, p, mlp, rnd=_same):
+def route_gaps(x, w_router, router: dict):
+    """Per token how far the last choice's logit lies above the best one that is not chosen (None: all are chosen)."""
+    if router["top"] == router["experts"]:
+        return None
+    z = torch.sort(x @ w_router.T, dim=1, descending=True).values
+    return z[:, router["top"] - 1] - z[:, router["top"]]
+
+
+def expert_mlp(x, w, p, mlp, rnd=_same, swapped=()):
     out = torch.zeros_like(x)
-    for t, picks in enumerate(route(x, w[p + "router"], mlp["router"])):
+    for t, picks in enumerate(route(x, w[p + "router"], mlp["router"], swapped)):
         for e, wt in picks:
             h = rnd(wt * x[t])
             a = silu(w[f"{p}e{e}.gate"] @ h) * (w[f"{p}e{e}.up"] @ h)
@@ -184,9 +197,10 @@ def expert_mlp(x, w, p, mlp, rnd=_same):
     return out
 
 
-def forward(config: dict, weights: dict, tokens, return_layers: bool = False, rnd=_same):
+def forward(config: dict, weights: dict, tokens, return_layers: bool = False, rnd=_same, swapped=(), gaps=None):
     """Logits [n, vocab] of a whole sequence (and the residual stream after every layer).  rnd: applied to what a
-    16-bit engine would store in 16 bits (what a matrix product reads, cached rows); the identity by default."""
+    16-bit engine would store in 16 bits (what a matrix product reads, cached rows); the identity by default.  swapped:
+    (layer, token) pairs whose router takes its closest call the other way; gaps: a dict that takes the routers' gaps by layer."""
     w = {k: (v.to(F64) if v.is_floating_point() else v) for k, v in weights.items()}
     eps = float(config["norm"]["eps"])
     x = w["embed"][torch.as_tensor(tokens, dtype=torch.long)]
@@ -208,7 +222,9 @@ def forward(config: dict, weights: dict, tokens, return_layers: bool = False, rn
         mlp = layer.get("mlp")
         if mlp is not None:
             h = rnd(x)
-            upd = (expert_mlp(h, w, p + "mlp.", mlp, rnd) if mlp["kind"] == "moe"
+            if mlp["kind"] == "moe" and gaps is not None:
+                gaps[i] = route_gaps(h, w[p + "mlp.router"], mlp["router"])
+            upd = (expert_mlp(h, w, p + "mlp.", mlp, rnd, [t for n, t in swapped if n == i]) if mlp["kind"] == "moe"
                    else relu2_mlp(h, w[p + "mlp.up"], w[p + "mlp.down"], rnd))
             x = x + w[p + "ls2"] * ln(upd, w[p + "norm2"], w[p + "norm2.b"], eps)
         streams.append(x.clone())
