@@ -1266,12 +1266,13 @@ def fugavik_kernels(z: dict, T: int, peaks: dict) -> dict:
     w_uk = (torch.randn(H, e, L, device=dev) / e ** 0.5).to(bf)
     w_uv = (torch.randn(H, L, ev, device=dev) / L ** 0.5).to(bf)
     ov = torch.empty(T, H * ev, dtype=bf, device=dev)
-    note("queries onto the latent, a product per head (nikonex)", timed(lambda: ops.heads_linear(down, e, w_uk, qf, L), flush),
+    uk, uv = (w_uk, w_uk.transpose(1, 2).contiguous()), (w_uv, w_uv.transpose(1, 2).contiguous())
+    note("queries onto the latent, a product per head (nikonex)", timed(lambda: rt.heads_linear(down[:, :H * e], e, uk, qf, L), flush),
          flops=2.0 * T * H * e * L, nbytes=T * H * (e + L) * 2 + w_uk.numel() * 2)
-    note("values from the latent, a product per head (nikonex)", timed(lambda: ops.heads_linear(of, L, w_uv, ov, ev), flush),
+    note("values from the latent, a product per head (nikonex)", timed(lambda: rt.heads_linear(of, L, uv, ov, ev), flush),
          flops=2.0 * T * H * L * ev, nbytes=T * H * (L + ev) * 2 + w_uv.numel() * 2)
     note("values from the latent, a product per head, times the head's gate", timed(
-        lambda: ops.heads_linear(of, L, w_uv, ov, ev, gate=down[:, H * e + L:]), flush),
+        lambda: rt.heads_linear(of, L, uv, ov, ev, gate=down[:, H * e + L:]), flush),
         flops=2.0 * T * H * L * ev, nbytes=T * H * (L + ev) * 2 + w_uv.numel() * 2)
     # the delta rule beside retention's recurrence at equal heads and sizes, with its convolution and the heads' norm
     RH, G, dk, dv = z["delta_heads"], z["delta_kv"], z["delta_dim"], z["delta_v"]

@@ -58,6 +58,7 @@ struct Params2 {
     // parts, part s written to the slice s of the output, split_stride elements apart, as C[token][weight row].
     int n_split, kb_per_split;
     long long split_stride;
+    int out_act = 0;       // not DUAL, bfloat16 out: 1 = C is max(z, 0)^2 of the product
     int gate_act = 0;      // DUAL: what the gate goes through, 0 SiLU, 1 tanh-GELU
 };
 
@@ -351,6 +352,13 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant
                 } else {
                     tc::tmem_ld32(taddr, r);
                     tc::tmem_ld_wait();
+                    if (std::is_same<TO, bf16>::value && p.out_act) {
+#pragma unroll
+                        for (int q = 0; q < 32; ++q) {
+                            const float z = fmaxf(__uint_as_float(r[q]), 0.f);
+                            r[q] = __float_as_uint(z * z);
+                        }
+                    }
                 }
                 const int j0 = tn * ACC_N + c0;
                 if (i < p.M && j0 < p.N) {
@@ -481,8 +489,9 @@ int launch2(const CUtensorMap& ma, const CUtensorMap& mw, const Params2& p, cuda
 // stride lda; W: bfloat16, row stride ldw; C of c_dtype (bfloat16 or float32), row stride ldc.
 // Strides and K multiples of 8 elements, pointers 16-byte aligned, else ODIN_ERR_UNSUPPORTED.
 // accumulate (float32 C only): C += A W^T, each element read once and written once by the thread that holds its sum.
+// act (bfloat16 C only): 1 = C is max(z, 0)^2 of the product, formed as the sums are read back.
 extern "C" int odin_gemm_tc2(const void* A, const void* W, void* C, int c_dtype, int M, int N, int K, long long lda,
-                             long long ldw, long long ldc, int accumulate, void* stream) {
+                             long long ldw, long long ldc, int accumulate, int act, void* stream) {
     if (M <= 0 || N <= 0) return 0;
     if (K <= 0) return ODIN_ERR_BAD_ARG;
     if ((lda % 8) || (ldw % 8) || (K % 8) || (((uintptr_t)A) & 15) || (((uintptr_t)W) & 15)) return ODIN_ERR_UNSUPPORTED;
@@ -495,6 +504,8 @@ extern "C" int odin_gemm_tc2(const void* A, const void* W, void* C, int c_dtype,
     p.n_split = 1; p.kb_per_split = p.kb_total; p.split_stride = 0;
     if (accumulate && c_dtype != ODIN_F32) return ODIN_ERR_BAD_ARG;
     p.accumulate = accumulate ? 1 : 0;
+    if (act < 0 || act > 1 || (act && c_dtype != ODIN_BF16)) return ODIN_ERR_BAD_ARG;
+    p.out_act = act;
     p.error = error_flag2();
     CUtensorMap ma, mw;
     int rc;

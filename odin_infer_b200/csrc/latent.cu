@@ -13,7 +13,7 @@
 //
 // All arithmetic is 32-bit.  Every output element is one sum in an order that the sizes fix (k ascending in one
 // thread; a row's sum of squares by the block's fixed tree), so a token's values do not depend on the batch.
-#include "common.cuh"
+#include "head_gate.cuh"
 
 #define LP_THREADS 128
 
@@ -112,21 +112,6 @@ extern "C" int odin_latent_prep(const void* down, int in_dtype, int n_split, lon
 #define HL_TOK 8
 #define HL_PRE 32
 
-struct HeadGate {
-    const void* p;             // null: no gate
-    int is_bf16, n_split;
-    long long split_stride, row_stride;
-    __device__ __forceinline__ float factor(int t, int h) const {
-        if (p == nullptr) return 1.0f;
-        float z = 0.f;
-        for (int s = 0; s < n_split; ++s) {
-            const size_t at = (size_t)s * split_stride + (size_t)t * row_stride + h;
-            z += is_bf16 ? __bfloat162float(((const bf16*)p)[at]) : ((const float*)p)[at];
-        }
-        return 1.0f / (1.0f + expf(-z));
-    }
-};
-
 template <typename TA>
 __device__ __forceinline__ float sum_parts(const TA* __restrict__ a, size_t at, int n_split, size_t split_stride) {
     float v = to_f32(a[at]);
@@ -147,9 +132,15 @@ heads_linear_kernel(const TA* __restrict__ a, int a_splits, size_t a_ss, size_t 
     const TW* wh = w + (size_t)h * K * N + n;
     TW cur[HL_PRE], nxt[HL_PRE];
     auto fetch = [&](TW (&dst)[HL_PRE], int k0) {
+        if (n >= N) return;
+        if (k0 + HL_PRE <= K) {
 #pragma unroll
-        for (int j = 0; j < HL_PRE; ++j)
-            if (n < N && k0 + j < K) dst[j] = wh[(size_t)(k0 + j) * N];
+            for (int j = 0; j < HL_PRE; ++j) dst[j] = wh[(size_t)(k0 + j) * N];
+        } else {
+#pragma unroll
+            for (int j = 0; j < HL_PRE; ++j)
+                if (k0 + j < K) dst[j] = wh[(size_t)(k0 + j) * N];
+        }
     };
     fetch(cur, 0);
     pdl_wait();
@@ -181,23 +172,26 @@ heads_linear_kernel(const TA* __restrict__ a, int a_splits, size_t a_ss, size_t 
     float acc[HL_TOK];
 #pragma unroll
     for (int u = 0; u < HL_TOK; ++u) acc[u] = 0.f;
-    for (int k0 = 0; k0 < K; k0 += HL_PRE) {
+    auto take = [&](int k, TW wk) {
+        const float wv = to_f32(wk);
+        const float4 a0 = *reinterpret_cast<const float4*>(&as[k * HL_TOK]);
+        const float4 a1 = *reinterpret_cast<const float4*>(&as[k * HL_TOK + 4]);
+        acc[0] = fmaf(wv, a0.x, acc[0]); acc[1] = fmaf(wv, a0.y, acc[1]);
+        acc[2] = fmaf(wv, a0.z, acc[2]); acc[3] = fmaf(wv, a0.w, acc[3]);
+        acc[4] = fmaf(wv, a1.x, acc[4]); acc[5] = fmaf(wv, a1.y, acc[5]);
+        acc[6] = fmaf(wv, a1.z, acc[6]); acc[7] = fmaf(wv, a1.w, acc[7]);
+    };
+    int k0 = 0;
+    for (; k0 + HL_PRE <= K; k0 += HL_PRE) {
         fetch(nxt, k0 + HL_PRE);
 #pragma unroll
-        for (int j = 0; j < HL_PRE; ++j) {
-            if (k0 + j < K) {
-                const float wv = to_f32(cur[j]);
-                const float4 a0 = *reinterpret_cast<const float4*>(&as[(k0 + j) * HL_TOK]);
-                const float4 a1 = *reinterpret_cast<const float4*>(&as[(k0 + j) * HL_TOK + 4]);
-                acc[0] = fmaf(wv, a0.x, acc[0]); acc[1] = fmaf(wv, a0.y, acc[1]);
-                acc[2] = fmaf(wv, a0.z, acc[2]); acc[3] = fmaf(wv, a0.w, acc[3]);
-                acc[4] = fmaf(wv, a1.x, acc[4]); acc[5] = fmaf(wv, a1.y, acc[5]);
-                acc[6] = fmaf(wv, a1.z, acc[6]); acc[7] = fmaf(wv, a1.w, acc[7]);
-            }
-        }
+        for (int j = 0; j < HL_PRE; ++j) take(k0 + j, cur[j]);
 #pragma unroll
         for (int j = 0; j < HL_PRE; ++j) cur[j] = nxt[j];
     }
+#pragma unroll
+    for (int j = 0; j < HL_PRE; ++j)
+        if (k0 + j < K) take(k0 + j, cur[j]);
 #pragma unroll
     for (int u = 0; u < HL_TOK; ++u)
         if (t0 + u < T) out[(size_t)(t0 + u) * o_rs + (size_t)h * o_hs + n] = from_f32<TO>(acc[u] * factors[u]);

@@ -18,6 +18,7 @@
 #include <mutex>
 #include <unordered_map>
 
+#include "head_gate.cuh"
 #include "tc_common.cuh"
 
 namespace {
@@ -167,6 +168,12 @@ struct GroupedParams {
     int stages;            // length of the ring of stages (2: two CTAs share an SM; 4: few CTAs, each with more in flight)
     const int* tile_expert;
     int* error;
+    // A product per head (tile_expert null): blockIdx.z is the head, which stands in for the expert; row tiles are tiles of
+    // tokens, a head's input columns start at head * a_hs of the token's row and its output columns at head * o_hs, and
+    // its outputs are multiplied by the head's gate.
+    int rows;
+    long long a_hs, o_hs;
+    HeadGate gate;
 };
 
 // DUAL: two accumulators of BN columns (gate, up), two weight boxes of BN rows a stage.  Plain: one accumulator of
@@ -219,7 +226,9 @@ moe_grouped_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_const
     }
     pdl_wait();   // the plan, the sorted rows and the output's memory belong to earlier kernels until here
     const int tile_m = blockIdx.y, tile_n = blockIdx.x;
-    const int e = p.tile_expert[tile_m];
+    const bool per_head = p.tile_expert == nullptr;
+    const int e = per_head ? (int)blockIdx.z : p.tile_expert[tile_m];
+    const int a_x0 = per_head ? (int)(e * p.a_hs) : 0;
     if (e < 0) return;   // a tile of places that no expert's rows reach (the whole CTA leaves, nothing is held yet)
     if (warp == 1) tc::tmem_alloc(tmem_slot, C::TMEM_COLS);
     tc::fence_before_sync();
@@ -237,7 +246,7 @@ moe_grouped_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_const
                 if (!tc::mbar_wait(&empty[stage], phase ^ 1, abort_flag)) { ok = false; break; }
                 uint8_t* sa = smem + stage * C::STAGE;
                 tc::mbar_expect_tx(&full[stage], C::STAGE);
-                tc::tma_load_2d(sa, &map_a, kb * BK, tile_m * BM, &full[stage]);
+                tc::tma_load_2d(sa, &map_a, a_x0 + kb * BK, tile_m * BM, &full[stage]);
                 if (DUAL) {   // two boxes of BN rows: the gate rows and, N rows further, the up rows
                     tc::tma_load_2d(sa + C::STAGE_A, &map_w, kb * BK, w_row0, &full[stage]);
                     tc::tma_load_2d(sa + C::STAGE_A + C::STAGE_B / 2, &map_w, kb * BK, w_row0 + p.N, &full[stage]);
@@ -279,7 +288,9 @@ moe_grouped_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_const
         if (tc::mbar_wait(acc_full, 0, abort_flag)) {
             tc::fence_after_sync();
             const size_t i = (size_t)tile_m * BM + quarter * 32 + lane;   // the place; every place of a tile exists
-            TO* out = reinterpret_cast<TO*>(p.out) + i * p.ldc;
+            TO* out = reinterpret_cast<TO*>(p.out) + i * p.ldc + (per_head ? (size_t)e * p.o_hs : 0);
+            const bool stored = !per_head || (int)i < p.rows;
+            const float factor = (per_head && stored) ? p.gate.factor((int)i, e) : 1.0f;
 #pragma unroll 1
             for (int c0 = 0; c0 < TILE_N; c0 += 32) {
                 uint32_t r[32];
@@ -294,13 +305,17 @@ moe_grouped_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_const
                 } else {
                     tc::tmem_ld32(taddr, r);
                     tc::tmem_ld_wait();
+                    if (per_head) {
+#pragma unroll
+                        for (int q = 0; q < 32; ++q) r[q] = __float_as_uint(__uint_as_float(r[q]) * factor);
+                    }
                     if (p.act != 0) {
 #pragma unroll
                         for (int q = 0; q < 32; ++q) r[q] = __float_as_uint(act_alone(p.act, __uint_as_float(r[q])));
                     }
                 }
                 const int j0 = tile_n * TILE_N + c0;
-                if (j0 < p.N) {
+                if (j0 < p.N && stored) {
                     const int n = min(32, p.N - j0);
                     if (sizeof(TO) == 4) {
                         float* dst = reinterpret_cast<float*>(out) + j0;
@@ -329,6 +344,7 @@ moe_grouped_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_const
                         }
                     }
                 }
+                __syncwarp();   // rows beyond the last token store nothing
             }
         }
     }
@@ -395,7 +411,7 @@ int sm_count() {
 }
 
 template <bool DUAL, typename TO>
-int launch_grouped(const CUtensorMap& ma, const CUtensorMap& mw, GroupedParams p, int tiles_m, cudaStream_t s) {
+int launch_grouped(const CUtensorMap& ma, const CUtensorMap& mw, GroupedParams p, int tiles_m, cudaStream_t s, int heads = 1) {
     using C = GCfg;
     static bool configured = false;
     if (!configured) {
@@ -405,12 +421,12 @@ int launch_grouped(const CUtensorMap& ma, const CUtensorMap& mw, GroupedParams p
         configured = true;
     }
     const int tile_n = DUAL ? BN : 2 * BN;
-    const dim3 grid((unsigned)((p.N + tile_n - 1) / tile_n), (unsigned)tiles_m);
+    const dim3 grid((unsigned)((p.N + tile_n - 1) / tile_n), (unsigned)tiles_m, (unsigned)heads);
     // Few CTAs (a step of few tokens: the weights stream once, and about half of the grid's row tiles are places that no
     // expert's rows reach, whose CTAs leave at once; measured at 138 working CTAs: 37.5 us against 43.6): a ring of four
     // stages, so that enough is in flight; many CTAs: two stages, and two CTAs share an SM, one's epilogue beside the
     // other's products.  The number of CTAs follows from the shapes alone.
-    p.stages = ((long long)grid.x * grid.y <= 2LL * sm_count()) ? C::MAX_STAGES : 2;
+    p.stages = ((long long)grid.x * grid.y * grid.z <= 2LL * sm_count()) ? C::MAX_STAGES : 2;
     odin_launch(moe_grouped_kernel<DUAL, TO>, grid, dim3(192), (size_t)C::smem(p.stages), s, ma, mw, p);
     ODIN_LAUNCH_CHECK();
     return 0;
@@ -467,7 +483,7 @@ extern "C" int odin_moe_grouped(const void* a, long long lda, const void* w, lon
     int rc;
     if ((rc = make_map(&ma, a, places, K, lda, BM))) return rc;
     if ((rc = make_map(&mw, w, (long long)n_experts * rows_per_expert, K, ldw, dual ? BN : 2 * BN))) return rc;
-    GroupedParams p;
+    GroupedParams p = {};
     p.out = out; p.ldc = ldc; p.N = N; p.K = K; p.rows_per_expert = rows_per_expert; p.act = act; p.stages = 2;
     p.tile_expert = tile_expert;
     p.error = error_flag();
@@ -478,6 +494,26 @@ extern "C" int odin_moe_grouped(const void* a, long long lda, const void* w, lon
         return launch_grouped<false, bf16>(ma, mw, p, places / BM, s);
     }
     return launch_grouped<false, float>(ma, mw, p, places / BM, s);
+}
+
+// A product per head for many tokens: out[t, h * o_hs + n] = sigmoid(gate[t, h]) * sum_k a[t, h * a_hs + k] w[h][n][k].
+// a: [T, a_cols] bfloat16 of row stride lda; w: [H][N][K] bfloat16, K a multiple of 64; out: bfloat16 of row stride ldc.
+extern "C" int odin_heads_linear_tc(const void* a, long long lda, long long a_hs, int a_cols, const void* w, void* out,
+                                    long long ldc, long long o_hs, int T, int H, int N, int K, const void* gate,
+                                    int gate_dtype, int gate_splits, long long gate_ss, long long gate_rs, void* stream) {
+    if (T <= 0) return 0;
+    if (H <= 0 || H > 65535 || N <= 0 || K <= 0 || (gate != nullptr && gate_splits < 1)) return ODIN_ERR_BAD_ARG;
+    if ((lda % 8) || (a_hs % 8) || (K % 64) || (((uintptr_t)a) & 15) || (((uintptr_t)w) & 15) || T > 65535 * BM) return ODIN_ERR_UNSUPPORTED;
+    CUtensorMap ma, mw;
+    int rc;
+    if ((rc = make_map(&ma, a, T, a_cols, lda, BM))) return rc;
+    if ((rc = make_map(&mw, w, (long long)H * N, K, K, 2 * BN))) return rc;
+    GroupedParams p = {};
+    p.out = out; p.ldc = ldc; p.N = N; p.K = K; p.rows_per_expert = N; p.stages = 2;
+    p.error = error_flag();
+    p.rows = T; p.a_hs = a_hs; p.o_hs = o_hs;
+    p.gate = HeadGate{gate, gate_dtype == ODIN_BF16, gate_splits, gate_ss, gate_rs};
+    return launch_grouped<false, bf16>(ma, mw, p, (T + BM - 1) / BM, (cudaStream_t)stream, H);
 }
 
 extern "C" int odin_moe_tc_error() {

@@ -811,6 +811,34 @@ def heads_linear(a: torch.Tensor, a_head_stride: int, w: torch.Tensor, out: torc
         _stream()), "heads_linear")
 
 
+def heads_linear_tc_supported(a: torch.Tensor, a_head_stride: int, w: torch.Tensor) -> bool:
+    """Shapes and types that the tensor-core product per head takes (w: [H, N, K])"""
+    K = w.shape[2]
+    return (a.dim() == 2 and a.dtype == w.dtype == torch.bfloat16 and a.stride(1) == 1 and K % 64 == 0
+            and a_head_stride % 8 == 0 and a.stride(0) % 8 == 0 and a.data_ptr() % 16 == 0 and w.is_contiguous())
+
+
+def heads_linear_tc(a: torch.Tensor, a_head_stride: int, w: torch.Tensor, out: torch.Tensor, out_head_stride: int,
+                    gate: torch.Tensor | None = None) -> None:
+    """`heads_linear` on the tcgen05 tensor cores, for many tokens: w is [H, N, K] (output channel before input channel),
+    a and out bfloat16."""
+    H, N, K = w.shape
+    T = a.shape[0]
+    if not heads_linear_tc_supported(a, a_head_stride, w):
+        raise KernelError("heads_linear_tc: bfloat16 rows of whole 16 bytes and K a multiple of 64")
+    assert out.dtype == torch.bfloat16 and out.stride(1) == 1 and out.shape[0] == T
+    assert a.shape[1] >= (H - 1) * a_head_stride + K and out.shape[1] >= (H - 1) * out_head_stride + N
+    g_split, g_ss, g_rs = (1, 0, 0)
+    if gate is not None:
+        assert tuple(gate.shape[-2:]) == (T, H)
+        g_split, g_ss, g_rs = _parts_view(gate)
+    _check(_fn("moe_tc", "odin_heads_linear_tc")(
+        _ptr(a), c_longlong(a.stride(0)), c_longlong(a_head_stride), c_int(a.shape[1]), _ptr(w), _ptr(out),
+        c_longlong(out.stride(0)), c_longlong(out_head_stride), c_int(T), c_int(H), c_int(N), c_int(K), _ptr(gate),
+        c_int(dtype_code(gate.dtype) if gate is not None else 0), c_int(g_split), c_longlong(g_ss), c_longlong(g_rs),
+        _stream()), "heads_linear_tc")
+
+
 def rope_heads(src: torch.Tensor, src_head_stride: int, dst: torch.Tensor, dst_head_stride: int, n_heads: int, width: int,
                rot: int, pairs: bool, cos: torch.Tensor, sin: torch.Tensor, tok_pos: torch.Tensor, scale: float = 1.0,
                scale_from_head: int | None = None) -> None:
@@ -904,9 +932,9 @@ def gemm_tc_swiglu(a: torch.Tensor, w_gate_up: torch.Tensor, out: torch.Tensor, 
         c_int(GATE_ACTS[activation]), _stream()), "gemm_tc_swiglu")
 
 
-def gemm_tc2(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate: bool = False) -> None:
+def gemm_tc2(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate: bool = False, relu2: bool = False) -> None:
     """out = a[M, K] @ w[N, K]^T on pairs of SMs (tcgen05 cta_group::2, tiles of 256 x 256): for many tokens.
-    accumulate: out (float32) += the product."""
+    accumulate: out (float32) += the product.  relu2: out (bfloat16) = max(z, 0)^2 of the product."""
     M, K = a.shape
     N = w.shape[0]
     if not gemm_tc_supported(a, w):
@@ -915,7 +943,7 @@ def gemm_tc2(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, accumulate: bo
     _check(_fn("gemm_tc", "odin_gemm_tc2")(
         _ptr(a), _ptr(w), _ptr(out), c_int(dtype_code(out.dtype)), c_int(M), c_int(N), c_int(K),
         c_longlong(a.stride(0)), c_longlong(w.stride(0)), c_longlong(out.stride(0)), c_int(1 if accumulate else 0),
-        _stream()), "gemm_tc2")
+        c_int(1 if relu2 else 0), _stream()), "gemm_tc2")
 
 
 def gemm_tc2_wide(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, n_split: int = 1) -> None:

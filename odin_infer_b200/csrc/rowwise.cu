@@ -710,6 +710,99 @@ combine_add_kernel(float* __restrict__ x, CombineArgs a, CombineNorm post, Combi
     }
 }
 
+// The same for one term without a norm or a number per row of its own, a row of up to 1,024 NV elements (the width a multiple of
+// four, everything 16-byte aligned): the row stays in registers, its loads go out together, and a sum over the row costs one
+// barrier (every warp's share goes to a place of its own, and every thread adds the eight shares in their order).
+template <typename TD, typename TO, int NV>
+__global__ void __launch_bounds__(ROW_THREADS)
+combine_one_kernel(float* __restrict__ x, const TD* __restrict__ delta, int n_split, size_t split_stride, float scale,
+                   CombineNorm post, CombineNorm next, TO* __restrict__ out, const int* __restrict__ rows,
+                   const int* __restrict__ tok_seq, int d) {
+    __shared__ __align__(16) float shares[4][ROW_THREADS / 32];
+    pdl_trigger();
+    const int r = rows != nullptr ? rows[blockIdx.x] : blockIdx.x;
+    const bool real = tok_seq == nullptr || tok_seq[r] >= 0;
+    pdl_wait();
+    if (!real) return;
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    int n_sums = 0;
+    auto row_sum = [&](float v) {
+        float* sh = shares[n_sums++];
+        v = warp_sum(v);
+        if (lane == 0) sh[warp] = v;
+        __syncthreads();
+        const float4 a = ld4(sh), b = ld4(sh + 4);
+        return ((a.x + a.y) + (a.z + a.w)) + ((b.x + b.y) + (b.z + b.w));
+    };
+    auto statistics = [&](const float4 (&v)[NV], const CombineNorm& nm, float& mean, float& rs) {
+        float s = 0.f;
+        mean = 0.f;
+        if (nm.center) {
+#pragma unroll
+            for (int i = 0; i < NV; ++i) s += (v[i].x + v[i].y) + (v[i].z + v[i].w);   // zeros beyond the row
+            mean = row_sum(s) / (float)d;
+            s = 0.f;
+        }
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+            if ((threadIdx.x + i * ROW_THREADS) * 4 < d) {
+                const float a = v[i].x - mean, b = v[i].y - mean, c = v[i].z - mean, e = v[i].w - mean;
+                s += (a * a + b * b) + (c * c + e * e);
+            }
+        rs = 1.0f / sqrtf(row_sum(s) / (float)d + nm.eps);
+    };
+    auto normed = [&](const float4& v, const CombineNorm& nm, int j, float mean, float rs) {
+        const float4 w = nm.w.at4(j);
+        float4 y = make_float4(w.x * (rs * (v.x - mean)), w.y * (rs * (v.y - mean)), w.z * (rs * (v.z - mean)), w.w * (rs * (v.w - mean)));
+        if (nm.b.p != nullptr) {
+            const float4 b = nm.b.at4(j);
+            y.x += b.x; y.y += b.y; y.z += b.z; y.w += b.w;
+        }
+        return y;
+    };
+    float* xr = x + (size_t)r * d;
+    float4 xv[NV], u[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int j = (threadIdx.x + i * ROW_THREADS) * 4;
+        xv[i] = u[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (j < d) xv[i] = ld4(xr + j);
+    }
+    for (int s = 0; s < n_split; ++s) {
+#pragma unroll
+        for (int i = 0; i < NV; ++i) {
+            const int j = (threadIdx.x + i * ROW_THREADS) * 4;
+            if (j < d) {
+                const float4 v = ld4(delta + (size_t)s * split_stride + (size_t)r * d + j);
+                u[i].x += v.x; u[i].y += v.y; u[i].z += v.z; u[i].w += v.w;
+            }
+        }
+    }
+    if (scale != 1.0f) {
+#pragma unroll
+        for (int i = 0; i < NV; ++i) { u[i].x *= scale; u[i].y *= scale; u[i].z *= scale; u[i].w *= scale; }
+    }
+    float mean = 0.f, rs = 1.0f;
+    if (post.w.p != nullptr) statistics(u, post, mean, rs);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int j = (threadIdx.x + i * ROW_THREADS) * 4;
+        if (j >= d) continue;
+        const float4 y = post.w.p != nullptr ? normed(u[i], post, j, mean, rs) : u[i];
+        xv[i].x += y.x; xv[i].y += y.y; xv[i].z += y.z; xv[i].w += y.w;
+        if (rows == nullptr) st4(xr + j, xv[i]);
+    }
+    if (out == nullptr) return;
+    mean = 0.f;
+    if (next.w.p != nullptr) statistics(xv, next, mean, rs);
+    TO* orow = out + (size_t)blockIdx.x * d;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int j = (threadIdx.x + i * ROW_THREADS) * 4;
+        if (j < d) st4(orow + j, next.w.p != nullptr ? normed(xv[i], next, j, mean, rs) : xv[i]);
+    }
+}
+
 extern "C" int odin_combine_add(float* x, int n_terms, const void* const* ptrs, const int* dtypes, const int* n_splits,
                                 const long long* split_strides, const float* scales, const float* const* row_scales,
                                 const void* const* norm_ws, const int* norm_w_dtypes, const float* norm_eps,
@@ -738,6 +831,26 @@ extern "C" int odin_combine_add(float* x, int n_terms, const void* const* ptrs, 
     cudaStream_t s = (cudaStream_t)stream;
     const CombineNorm post{VecRef{post_w, post_w_dtype == ODIN_BF16}, VecRef{post_b, post_b_dtype == ODIN_BF16}, post_eps, post_center};
     const CombineNorm next{VecRef{next_w, next_w_dtype == ODIN_BF16}, VecRef{next_b, next_b_dtype == ODIN_BF16}, next_eps, next_center};
+    if (vec && x != nullptr && n_terms == 1 && norm_ws[0] == nullptr && row_scales[0] == nullptr && d <= 4 * 1024) {
+        const int nv = d <= 1024 ? 1 : d <= 2048 ? 2 : 4;
+#define ONE(TD, TO, NV)                                                                                              \
+    odin_launch(combine_one_kernel<TD, TO, NV>, dim3(n_rows), dim3(ROW_THREADS), 0, s, x, (const TD*)ptrs[0],         \
+                n_splits[0], (size_t)split_strides[0], scales[0], post, next, (TO*)out, rows, tok_seq, d)
+#define ONE_NV(TD, TO)                                                                                               \
+    do {                                                                                                             \
+        if (nv == 1) ONE(TD, TO, 1);                                                                                 \
+        else if (nv == 2) ONE(TD, TO, 2);                                                                            \
+        else ONE(TD, TO, 4);                                                                                         \
+    } while (0)
+        const bool out_bf16 = out != nullptr && out_dtype == ODIN_BF16;
+        if (out != nullptr && out_dtype != ODIN_BF16 && out_dtype != ODIN_F32) return ODIN_ERR_UNSUPPORTED;
+        if (dtypes[0] == ODIN_BF16) { if (out_bf16) ONE_NV(bf16, bf16); else ONE_NV(bf16, float); }
+        else { if (out_bf16) ONE_NV(float, bf16); else ONE_NV(float, float); }
+#undef ONE_NV
+#undef ONE
+        ODIN_LAUNCH_CHECK();
+        return 0;
+    }
 #define GO(TO)                                                                                                       \
     do {                                                                                                             \
         auto kern = vec ? combine_add_kernel<TO, true> : combine_add_kernel<TO, false>;                              \

@@ -52,6 +52,9 @@ WIDE_CHUNKS_MAX_TOKENS = int(os.environ.get("ODIN_WIDE_CHUNKS_MAX_TOKENS", "1024
 # shorter than the row kernels', although it launches three kernels more; at 192 rows half as long)
 MOE_GROUPED_FROM_ROWS = int(os.environ.get("ODIN_MOE_GROUPED_FROM", "32"))
 
+# from this many tokens on a product per head runs on the tensor cores
+HEADS_TC_FROM = 128
+
 # ring length of a product that shares the SM with a decode attention CTA (see Runtime.linear)
 LIGHT_STAGES = int(os.environ.get("ODIN_GEMM_LIGHT_STAGES", "5"))
 
@@ -226,9 +229,23 @@ class Runtime:
     def activated_linear(self, a: torch.Tensor, w: torch.Tensor, activation: str, params: torch.Tensor | None = None) -> torch.Tensor:
         """act(a W^T): a product followed by the activation kernel (which also adds the partial sums of a split product).
         activation: one of `ops.ACTIVATIONS`; params: its numbers, where it has any."""
-        act = self.empty(a.shape[0], w.shape[0])
+        M, N = a.shape[0], w.shape[0]
+        act = self.empty(M, N)
+        if (activation == "relu2" and self.dtype == torch.bfloat16 and M >= PAIR_MIN_TOKENS and N > 128 and ops.gemm_tc_supported(a, w)
+                and (M > WIDE_CHUNKS_MAX_TOKENS or (N + 255) // 256 >= self.n_sms // 2)):
+            # many tokens: the activation rides in the product's epilogue
+            ops.gemm_tc2(a, w, act, relu2=True)
+            return act
         ops.activation(self.linear(a, w, may_split=True), activation, act, params)
         return act
+
+    def heads_linear(self, a, a_head_stride: int, w, out: torch.Tensor, out_head_stride: int, gate=None) -> None:
+        """A product per head (see `ops.heads_linear`); w: the heads' matrices in both orders, ([H, K, N], [H, N, K]).  Many
+        bfloat16 tokens go to the tensor cores."""
+        if out.shape[0] >= HEADS_TC_FROM and self.dtype == torch.bfloat16 and ops.heads_linear_tc_supported(a, a_head_stride, w[1]):
+            ops.heads_linear_tc(a, a_head_stride, w[1], out, out_head_stride, gate)
+        else:
+            ops.heads_linear(a, a_head_stride, w[0], out, out_head_stride, gate)
 
     # ---- experts chosen per token ----------------------------------------
     def experts(self, h: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor,

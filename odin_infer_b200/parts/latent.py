@@ -83,16 +83,18 @@ class LatentAttention(Mixer):
                 self.q_norm, self.c_norm = self.q_norm.float(), self.c_norm.float()
         if self.sink_name is not None:
             self.sink = tensors[self.sink_name].to(torch.float32).contiguous()
-        # per head, input channel before output channel: W_uk of a head as it is stored, W_uv of a head transposed
-        self.w_uk = tensors.pop(n["uk"]).view(H, self.e, self.kv_rank).contiguous()
-        self.w_uv = tensors.pop(n["uv"]).view(H, self.ev, self.kv_rank).transpose(1, 2).contiguous()
+        # per head, (input channel before output channel, output before input): W_uk of a head is stored the first way, W_uv
+        # the second
+        uk, uv = tensors.pop(n["uk"]).view(H, self.e, self.kv_rank), tensors.pop(n["uv"]).view(H, self.ev, self.kv_rank)
+        self.w_uk = (uk.contiguous(), uk.transpose(1, 2).contiguous())
+        self.w_uv = (uv.transpose(1, 2).contiguous(), uv.contiguous())
         self._dummy = torch.zeros(1, 1, dtype=torch.float32, device=rt.device)
 
     def cache_request(self):
         return KVRequest(1, self.L, self.window, 0, 0, shared_kv=True)
 
     def kernel_groups(self):
-        return {"latent", "attention_plain", "gemm_plain"}
+        return {"latent", "moe_tc", "attention_plain", "gemm_plain"}
 
     def notes(self, rt):
         if rt.dtype != torch.bfloat16:
@@ -121,11 +123,11 @@ class LatentAttention(Mixer):
                         write_cache=step.writes_cache(entry))
         q = rt.linear(cq, self.w_uq) if self.q_rank else down[..., :n0]
         qf = rt.empty(T, H * L)
-        ops.heads_linear(q, e + r, self.w_uk, qf, L)
+        rt.heads_linear(q, e + r, self.w_uk, qf, L)
         if r:
             ops.rope_heads(q[:, e:], e + r, qf[:, self.kv_rank:], L, H, r, r, pairs, cos, sin, step.tok_pos)
         o = rt.empty(T, H * L)
         rt.attention(step, qf, o, H, 1, L, line, line, block_table, self.window, scale=self.scale, sink=self.sink)
         ov = rt.empty(T, H * self.ev)
-        ops.heads_linear(o, L, self.w_uv, ov, self.ev, gate=down[..., n1:] if self.gate_name is not None else None)
+        rt.heads_linear(o, L, self.w_uv, ov, self.ev, gate=down[..., n1:] if self.gate_name is not None else None)
         return rt.linear(ov, self.w_o, out_dtype=torch.float32, may_split=True, beside_attention=True)

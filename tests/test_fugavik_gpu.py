@@ -645,6 +645,26 @@ def test_product_per_head_with_partial_sums_and_a_gate(T, splits):
     close(out.view(T, H, N), want * torch.sigmoid(total[:, H * K + 11:])[:, :, None], 3e-6)
 
 
+@pytest.mark.parametrize("T", [128, 300])
+@pytest.mark.parametrize("H,K,N,pad", [(3, 64, 40, 0), (5, 128, 264, 24), (1, 192, 128, 8)])
+def test_product_per_head_on_the_tensor_cores(T, H, K, N, pad):
+    """Heads further apart than they are wide, output columns that are no whole tile, token counts that are none either, a
+    gate; the columns between the heads stay as they were."""
+    from odin_infer_b200.csrc import ops
+    torch.manual_seed(T + K)
+    a = torch.randn(T, H * (K + pad), device=DEV).to(torch.bfloat16)
+    w = (torch.randn(H, N, K, device=DEV) / K ** 0.5).to(torch.bfloat16)
+    gate = torch.randn(2, T, H + 3, device=DEV)
+    want = torch.einsum("thk,hnk->thn", a.double().view(T, H, K + pad)[:, :, :K], w.double())
+    for g in (None, gate[..., 3:]):
+        out = torch.full((T, H * (N + 2)), 7.0, dtype=torch.bfloat16, device=DEV)
+        ops.heads_linear_tc(a, K + pad, w, out, N + 2, gate=g)
+        got = out.view(T, H, N + 2)
+        close(got[:, :, :N], want if g is None else want * torch.sigmoid(gate.double().sum(0)[:, 3:])[:, :, None], 5e-3)
+        assert (got[:, :, N:] == 7.0).all()
+    ops.moe_tc_check()
+
+
 @pytest.mark.parametrize("T", [5, 300])
 @pytest.mark.parametrize("given_logits", [False, True])
 @pytest.mark.parametrize("E,top", [(8, 1), (5, 5), (1, 1), (40, 7)])
@@ -698,8 +718,8 @@ def test_experts_that_read_their_weight_times_the_input(dtype, tol, T, E, top, f
 
 
 @pytest.mark.parametrize("dtype,tol", [(torch.float32, 1e-5), (torch.bfloat16, 2e-2)])
-@pytest.mark.parametrize("T", [6, 150, 400])
-@pytest.mark.parametrize("width,ff", [(64, 96), (100, 36), (256, 512)])
+@pytest.mark.parametrize("T", [6, 150, 400, 1100])
+@pytest.mark.parametrize("width,ff", [(64, 96), (100, 36), (256, 520)])
 def test_dense_feed_forward_with_relu_squared(dtype, tol, T, width, ff):
     from odin_infer_b200.parts import PartSpec, build_part
     rt = runtime(dtype)
@@ -711,7 +731,7 @@ def test_dense_feed_forward_with_relu_squared(dtype, tol, T, width, ff):
 
 
 @pytest.mark.parametrize("dtype,tol", [(torch.float32, 2e-6), (torch.bfloat16, 1e-2)])
-@pytest.mark.parametrize("d,rows", [(96, 9), (100, 3), (2048, 5), (33, 4)])
+@pytest.mark.parametrize("d,rows", [(96, 9), (100, 3), (1028, 4), (2048, 5), (33, 4), (4096, 2), (4100, 2)])
 def test_layer_norm_of_an_update_the_add_and_what_follows(dtype, tol, d, rows):
     """The kernel behind the blocks: partial sums far from zero mean, the update's layer norm with its scale, the add, and then
     the stream converted, a layer norm of it (also with gathered rows, which leave the stream alone) or nothing."""
