@@ -104,12 +104,19 @@ delta_rule_kernel(DeltaParams dp) {
     float* st = p.state + (size_t)slot * p.state_stride + (size_t)head * dk * p.dv + j;
     // no other kernel of a step touches this layer's state: it is fetched while the kernel before this one still runs
     f32x2 S[SL / 2];
+    const bool whole = owns && i0 + SL <= dk;   // every channel of this lane exists: its loads go out together
+    {
+        float v[SL];
+        const float* sr = st + (size_t)i0 * p.dv;
+        if (whole) {
 #pragma unroll
-    for (int i = 0; i < SL; i += 2) {
-        float v[2];
+            for (int i = 0; i < SL; ++i) v[i] = sr[(size_t)i * p.dv];
+        } else {
 #pragma unroll
-        for (int e = 0; e < 2; ++e) v[e] = (owns && i0 + i + e < dk) ? st[(size_t)(i0 + i + e) * p.dv] : 0.f;
-        S[i / 2] = pack2(v[0], v[1]);
+            for (int i = 0; i < SL; ++i) v[i] = (owns && i0 + i < dk) ? sr[(size_t)i * p.dv] : 0.f;
+        }
+#pragma unroll
+        for (int i = 0; i < SL; i += 2) S[i / 2] = pack2(v[i], v[i + 1]);
     }
     pdl_wait();
     float* out = p.o + (size_t)head * p.dv + j;
@@ -385,16 +392,20 @@ delta_chunk_prepare_kernel(DeltaParams dp, DeltaChunks c) {
 #pragma unroll 1
         for (int h0 = 0; h0 < DC_TOK; h0 += 32) {
             f32x2 x[16];                       // rows h0 + 2 i and h0 + 2 i + 1
+            if (is_k) {
 #pragma unroll
-            for (int i = 0; i < 16; ++i) {
-                float v[2];
-#pragma unroll
-                for (int e = 0; e < 2; ++e) {
-                    const int t = h0 + 2 * i + e;
-                    if (is_k) v[e] = Ks[t * ld + cc] * bg[t];
-                    else v[e] = (t < nt && cc < p.dv) ? vr[(size_t)t * p.v_stride] * beta[t] : 0.f;
+                for (int i = 0; i < 16; ++i) {
+                    const int t = h0 + 2 * i;
+                    x[i] = pack2(Ks[t * ld + cc] * bg[t], Ks[(t + 1) * ld + cc] * bg[t + 1]);
                 }
-                x[i] = pack2(v[0], v[1]);
+            } else {
+                float v[32];                   // all loads first (rows beyond the sequence read its last row, and beta is zero there)
+                const bool in = cc < p.dv;
+#pragma unroll
+                for (int t = 0; t < 32; ++t) v[t] = in ? __ldg(vr + (size_t)min(h0 + t, nt - 1) * p.v_stride) : 0.f;
+#pragma unroll
+                for (int i = 0; i < 16; ++i)
+                    x[i] = pack2(v[2 * i] * beta[h0 + 2 * i], v[2 * i + 1] * beta[h0 + 2 * i + 1]);
             }
             if (h0 > 0) {
 #pragma unroll 2
