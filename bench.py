@@ -790,13 +790,14 @@ def nikonex_kernels(z: dict, T: int, peaks: dict) -> dict:
     w_uk = (torch.randn(H, e, kvr, device=dev) / e ** 0.5).to(bf)
     w_uv = (torch.randn(H, kvr, ev, device=dev) / kvr ** 0.5).to(bf)
     qf = torch.empty(T, H * L, dtype=bf, device=dev)
-    note("queries onto the latent, a product per head", timed(lambda: ops.heads_linear(q, e + r, w_uk, qf, L), flush),
+    uk, uv = (w_uk, w_uk.transpose(1, 2).contiguous()), (w_uv, w_uv.transpose(1, 2).contiguous())
+    note("queries onto the latent, a product per head", timed(lambda: rt.heads_linear(q, e + r, uk, qf, L), flush),
          flops=2.0 * T * H * e * kvr, nbytes=T * H * (e + kvr) * 2 + w_uk.numel() * 2)
     note("queries' rotated part into the wide row", timed(lambda: ops.rope_heads(q[:, e:], e + r, qf[:, kvr:], L, H, r, r, True, cos, sin, pos), flush),
          nbytes=T * H * r * 4)
     o = torch.empty(T, H * L, dtype=bf, device=dev)
     ov = torch.empty(T, H * ev, dtype=bf, device=dev)
-    note("values from the latent, a product per head", timed(lambda: ops.heads_linear(o, L, w_uv, ov, ev), flush),
+    note("values from the latent, a product per head", timed(lambda: rt.heads_linear(o, L, uv, ov, ev), flush),
          flops=2.0 * T * H * kvr * ev, nbytes=T * H * (kvr + ev) * 2 + w_uv.numel() * 2)
     # attention: every head over one shared row of L elements, beside grouped-query attention
     win = z["window"]

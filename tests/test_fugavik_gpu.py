@@ -72,11 +72,11 @@ ODD = model(97, 100, 1e-6,
             (attn(3, 1, 20, 28, 0.22, rot=20, base=900.0, factor=0.5, v_mix=True), dense(52)),
             (dlt(6, 2, 33, 9, 5), moe(4, 1, 28)))
 # head sizes the tensor-core attention kernels take, widths the tensor-core products take
-FAST = model(512, 128, 1e-5,
+FAST = model(384, 128, 1e-5,
              (dlt(4, 2, 64, 128, 4), moe(12, 2, 64)),
              (attn(4, 2, 64, 64, 0.15, rot=64, base=1e4, factor=8.0, v_mix=True), dense(256)),
-             (lat(8, 64, 32, 128, 0.12), moe(8, 1, 128)),
-             (attn(2, 2, 128, 64, 0.1, rot=64, base=1e6, factor=2.0, v_mix=True), dense(192)),
+             (lat(8, 64, 32, 128, 0.12), moe(9, 1, 128)),
+             (attn(2, 2, 128, 64, 0.1, rot=64, base=1e6, factor=2.5, v_mix=True), dense(176)),
              (attn(8, 2, 64, 64, 0.15, rot=64, base=1e4, factor=8.0, v_mix=True), None),
              (dlt(2, 1, 128, 64, 4), dense(128)))
 CONFIGS = {"mixed": (MIXED, 3), "odd": (ODD, 5), "fast": (FAST, 7)}
