@@ -31,6 +31,8 @@ GROUPS = {
     "recurrent": ["recurrent.cu"],
     "delta_rule": ["delta_rule.cu"],
     "state_space": ["state_space.cu"],
+    "gated_unit": ["gated_unit.cu"],
+    "streams": ["streams.cu"],
     "moe": ["moe.cu"],
     "moe_tc": ["moe_tc.cu"],
     "latent": ["latent.cu"],

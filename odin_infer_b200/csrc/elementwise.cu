@@ -11,7 +11,7 @@
 // ---------------------------------------------------------------- embedding
 template <typename TW>
 __global__ void embed_kernel(const TW* __restrict__ table, const int* __restrict__ ids,
-                             float* __restrict__ out, int d, int V, float scale) {
+                             float* __restrict__ out, int d, int V, float scale, int copies) {
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x;
@@ -19,18 +19,23 @@ __global__ void embed_kernel(const TW* __restrict__ table, const int* __restrict
     const bool ok = (id >= 0 && id < V);
     const TW* row = table + (size_t)(ok ? id : 0) * d;
     float* o = out + (size_t)t * d;
-    for (int j = threadIdx.x; j < d; j += blockDim.x) o[j] = ok ? to_f32(row[j]) * scale : 0.f;
+    const size_t next = (size_t)gridDim.x * d;   // a residual of several streams starts with as many copies of the rows
+    for (int j = threadIdx.x; j < d; j += blockDim.x) {
+        const float v = ok ? to_f32(row[j]) * scale : 0.f;
+        for (int k = 0; k < copies; ++k) o[k * next + j] = v;
+    }
 }
 
 extern "C" int odin_embed(const void* table, int table_dtype, const int* ids, float* out,
-                          int T, int d, int V, float scale, void* stream) {
+                          int T, int d, int V, float scale, int copies, void* stream) {
     if (T <= 0) return 0;
+    if (copies < 1) return ODIN_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     const int threads = d >= 1024 ? 256 : 128;
     if (table_dtype == ODIN_BF16)
-        odin_launch(embed_kernel<bf16>, dim3(T), dim3(threads), 0, s, (const bf16*)table, ids, out, d, V, scale);
+        odin_launch(embed_kernel<bf16>, dim3(T), dim3(threads), 0, s, (const bf16*)table, ids, out, d, V, scale, copies);
     else if (table_dtype == ODIN_F32)
-        odin_launch(embed_kernel<float>, dim3(T), dim3(threads), 0, s, (const float*)table, ids, out, d, V, scale);
+        odin_launch(embed_kernel<float>, dim3(T), dim3(threads), 0, s, (const float*)table, ids, out, d, V, scale, copies);
     else
         return ODIN_ERR_UNSUPPORTED;
     ODIN_LAUNCH_CHECK();
@@ -46,15 +51,17 @@ __global__ void embed_pair_kernel(const TW* __restrict__ table, const TW* __rest
                                   const int* __restrict__ tok_seq, const int* __restrict__ seq_start,
                                   const int* __restrict__ seq_slots, int* __restrict__ state, size_t state_stride,
                                   int buckets, long long mul_prev, long long mul_cur, float* __restrict__ out, int d, int V,
-                                  float scale, int store) {
+                                  float scale, int store, int copies) {
     pdl_trigger();
     pdl_wait();
     const int t = blockIdx.x;
     const int seq = tok_seq[t];
     float* o = out + (size_t)t * d;
     const int id = ids[t];
+    const size_t next = (size_t)gridDim.x * d;
     if (seq < 0 || id < 0 || id >= V) {
-        for (int j = threadIdx.x; j < d; j += blockDim.x) o[j] = 0.f;
+        for (int j = threadIdx.x; j < d; j += blockDim.x)
+            for (int k = 0; k < copies; ++k) o[k * next + j] = 0.f;
         return;
     }
     const int before = t > seq_start[seq] ? ids[t - 1] + 1 : state[(size_t)seq_slots[seq] * state_stride];
@@ -66,7 +73,10 @@ __global__ void embed_pair_kernel(const TW* __restrict__ table, const TW* __rest
     if (before > 0) rowp = (((long long)(before - 1) * mul_prev + (long long)id * mul_cur) % buckets + buckets) % buckets;
     const TW* row = table + (size_t)id * d;
     const TW* prow = pair + (size_t)rowp * d;
-    for (int j = threadIdx.x; j < d; j += blockDim.x) o[j] = to_f32(row[j]) * scale + to_f32(prow[j]);
+    for (int j = threadIdx.x; j < d; j += blockDim.x) {
+        const float v = to_f32(row[j]) * scale + to_f32(prow[j]);
+        for (int k = 0; k < copies; ++k) o[k * next + j] = v;
+    }
 }
 
 __global__ void store_last_token_kernel(const int* __restrict__ ids, const int* __restrict__ seq_start,
@@ -83,18 +93,18 @@ __global__ void store_last_token_kernel(const int* __restrict__ ids, const int* 
 extern "C" int odin_embed_pair(const void* table, const void* pair, int table_dtype, const int* ids, const int* tok_seq,
                                const int* seq_start, const int* seq_slots, int* state, long long state_stride, int n_seqs,
                                int buckets, long long mul_prev, long long mul_cur, float* out, int T, int d, int V,
-                               float scale, int single_rows, void* stream) {
+                               float scale, int single_rows, int copies, void* stream) {
     if (T <= 0) return 0;
-    if (buckets <= 0 || n_seqs <= 0) return ODIN_ERR_BAD_ARG;
+    if (copies < 1 || buckets <= 0 || n_seqs <= 0) return ODIN_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
     const int threads = d >= 1024 ? 256 : 128;
     if (table_dtype == ODIN_BF16)
         odin_launch(embed_pair_kernel<bf16>, dim3(T), dim3(threads), 0, s, (const bf16*)table, (const bf16*)pair, ids, tok_seq,
-                    seq_start, seq_slots, state, (size_t)state_stride, buckets, mul_prev, mul_cur, out, d, V, scale, single_rows);
+                    seq_start, seq_slots, state, (size_t)state_stride, buckets, mul_prev, mul_cur, out, d, V, scale, single_rows, copies);
     else if (table_dtype == ODIN_F32)
         odin_launch(embed_pair_kernel<float>, dim3(T), dim3(threads), 0, s, (const float*)table, (const float*)pair, ids,
                     tok_seq, seq_start, seq_slots, state, (size_t)state_stride, buckets, mul_prev, mul_cur, out, d,
-                    V, scale, single_rows);
+                    V, scale, single_rows, copies);
     else
         return ODIN_ERR_UNSUPPORTED;
     ODIN_LAUNCH_CHECK();

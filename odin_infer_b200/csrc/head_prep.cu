@@ -33,6 +33,8 @@ struct VMix {
 // rotation, no weight; 3: RMSNorm over the whole q projection (all query heads of the token at once; likewise k) with weights
 // of that size, before the rotation.  vd: size of a value head (key and query heads have hd).
 // pairs: the rotation pairs element 2i with 2i + 1 instead of i with i + rot/2.
+// v_is_k: the projection holds no values; a key head's elements with their bias, before norm and rotation, are also its
+// value head's (vd == hd), and its warp writes both.
 template <typename TI, typename T>
 __global__ void __launch_bounds__(HP_WARPS * 32)
 head_prep_kernel(const TI* qkv, int n_split, size_t split_stride, T* q_out,  // may alias: no restrict
@@ -40,7 +42,7 @@ head_prep_kernel(const TI* qkv, int n_split, size_t split_stride, T* q_out,  // 
                  VecRef kw, int norm_mode, float eps, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                  int rot, int table_len, const int* __restrict__ tok_pos, const int* __restrict__ tok_seq,
                  const int* __restrict__ block_table, int bt_stride, T* __restrict__ k_cache,
-                 T* __restrict__ v_cache, int page_size, int write_kv, int pairs, VMix<T> vmix) {
+                 T* __restrict__ v_cache, int page_size, int write_kv, int pairs, int v_is_k, VMix<T> vmix) {
     __shared__ float buf[HP_WARPS][HP_MAX_HD];
     __shared__ float whole_ss[2][HP_WARPS];
     pdl_trigger();
@@ -48,7 +50,7 @@ head_prep_kernel(const TI* qkv, int n_split, size_t split_stride, T* q_out,  // 
     const int t = blockIdx.x;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int head = blockIdx.y * HP_WARPS + warp;
-    const int n_heads = Hq + 2 * Hkv;
+    const int n_heads = Hq + (v_is_k ? 1 : 2) * Hkv;
     const int seq = tok_seq[t];
     if (seq < 0) return;  // padding token (the whole CTA: it belongs to one token)
     if (norm_mode == 3) {
@@ -101,6 +103,10 @@ head_prep_kernel(const TI* qkv, int n_split, size_t split_stride, T* q_out,  // 
         if (bias.p != nullptr) v += bias.at((int)col0 + j);
         b[j] = v;
         ss += v * v;
+    }
+    if (is_k && v_is_k) {   // the same place of the value cache (dst is its key's place)
+        T* vdst = v_cache + (dst - k_cache);
+        for (int j = lane; j < n; j += 32) vdst[j] = from_f32<T>(b[j]);
     }
     if (is_v) {  // value head: stored as it is, or mixed with an earlier layer's
         const size_t at = ((size_t)t * Hkv + kvh) * vd;
@@ -350,15 +356,16 @@ extern "C" int odin_head_prep(const void* qkv, int in_dtype, int n_split, long l
                               const float* cos_t, const float* sin_t, int rot, int table_len,
                               const int* tok_pos, const int* tok_seq, const int* block_table, int bt_stride,
                               void* k_cache, void* v_cache, int page_size, int write_kv, int pairs, const void* v_first,
-                              void* v_keep, float v_lambda, void* stream) {
+                              void* v_keep, float v_lambda, int v_is_k, void* stream) {
     if (T <= 0) return 0;
+    if (v_is_k && (vd != hd || v_first != nullptr || v_keep != nullptr)) return ODIN_ERR_BAD_ARG;
     if (hd > HP_MAX_HD || hd <= 0 || vd > HP_MAX_HD || vd <= 0 || (rot & 1) || rot > hd || rot < 0 || n_split < 1 ||
         norm_mode < 0 || norm_mode > 3)
         return ODIN_ERR_UNSUPPORTED;
     const int has_norm = norm_mode == 1;
-    const bool plain_heads = bias == nullptr && norm_mode < 2 && vd == hd && !pairs;
+    const bool plain_heads = bias == nullptr && norm_mode < 2 && vd == hd && !pairs && !v_is_k;
     cudaStream_t s = (cudaStream_t)stream;
-    const int n_heads = Hq + 2 * Hkv;
+    const int n_heads = Hq + (v_is_k ? 1 : 2) * Hkv;
     dim3 grid(T, (n_heads + HP_WARPS - 1) / HP_WARPS);
     if (grid.y > 65535) return ODIN_ERR_UNSUPPORTED;
     VecRef qw{q_norm_w, w_dtype == ODIN_BF16}, kw{k_norm_w, w_dtype == ODIN_BF16};
@@ -396,7 +403,7 @@ extern "C" int odin_head_prep(const void* qkv, int in_dtype, int n_split, long l
     odin_launch(head_prep_kernel<TI, TT>, grid, dim3(HP_WARPS * 32), 0, s,                                           \
         (const TI*)qkv, n_split, (size_t)split_stride, (TT*)q_out, (size_t)q_out_stride, Hq, Hkv, hd, vd,           \
         (size_t)row_stride, bv, qw, kw, norm_mode, eps, cos_t, sin_t, rot, table_len, tok_pos, tok_seq, block_table,     \
-        (int)bt_stride, (TT*)k_cache, (TT*)v_cache, page_size, write_kv, pairs,                                      \
+        (int)bt_stride, (TT*)k_cache, (TT*)v_cache, page_size, write_kv, pairs, v_is_k,                              \
         VMix<TT>{(const TT*)v_first, (TT*)v_keep, v_lambda})
     if (in_dtype == ODIN_BF16 && dtype == ODIN_BF16) GO(bf16, bf16);
     else if (in_dtype == ODIN_F32 && dtype == ODIN_F32) GO(float, float);

@@ -7,7 +7,7 @@
 //   heads_linear   a product per head: out[t, h, n] = sum_k a[t, h, k] * w[h][k][n].  With w = W_uk of head h it
 //                  turns a head's unrotated query into a query over the cached latent (q . (W_uk c) = (W_uk^T q) . c),
 //                  with w = W_uv^T of head h the attention's output over the latent into the head's value, times
-//                  sigmoid(gate[t, h]) where the heads are gated.
+//                  sigmoid(gate[t, h]) where the heads are gated, or sigmoid(gate[t, h, n]) where every element is.
 //   rope_heads     rotation of the first `rot` elements of every head by the token's position, pairs (2i, 2i+1) or
 //                  (i, i + rot/2), the rest copied; an optional factor on the heads from a given one on.
 //
@@ -107,7 +107,7 @@ extern "C" int odin_latent_prep(const void* down, int in_dtype, int n_split, lon
 // out[t, h, n] = sum_k a[t, h, k] * w[h][k][n]; a: row stride a_rs, head stride a_hs; out likewise; w: [H][K][N].
 // grid (N tiles of HL_THREADS, H, token tiles of HL_TOK); a thread owns one n for HL_TOK tokens and adds over k ascending.
 // a may be 32-bit partial sums of a split product (a_splits of them, a_ss elements apart, added in order); gate (optional):
-// a number per token and head, itself possibly partial sums; the sum is multiplied by its sigmoid.
+// a number per token and head (or per token and output element), itself possibly partial sums; the sum is multiplied by its sigmoid.
 #define HL_THREADS 128
 #define HL_TOK 8
 #define HL_PRE 32
@@ -194,7 +194,7 @@ heads_linear_kernel(const TA* __restrict__ a, int a_splits, size_t a_ss, size_t 
         if (k0 + j < K) take(k0 + j, cur[j]);
 #pragma unroll
     for (int u = 0; u < HL_TOK; ++u)
-        if (t0 + u < T) out[(size_t)(t0 + u) * o_rs + (size_t)h * o_hs + n] = from_f32<TO>(acc[u] * factors[u]);
+        if (t0 + u < T) out[(size_t)(t0 + u) * o_rs + (size_t)h * o_hs + n] = from_f32<TO>(acc[u] * factors[u] * gate.element(t0 + u, h, n, N));
 }
 
 // Many tokens: a CTA takes 64 tokens by 64 output channels of one head, K in steps of 32 through shared memory, a thread
@@ -256,7 +256,7 @@ heads_linear_tiled_kernel(const TA* __restrict__ a, int a_splits, size_t a_ss, s
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int n = n0 + tx * 4 + j;
-            if (n < N) out[(size_t)t * o_rs + (size_t)h * o_hs + n] = from_f32<TO>(acc[i][j] * f);
+            if (n < N) out[(size_t)t * o_rs + (size_t)h * o_hs + n] = from_f32<TO>(acc[i][j] * f * gate.element(t, h, n, N));
         }
     }
 }
@@ -264,10 +264,10 @@ heads_linear_tiled_kernel(const TA* __restrict__ a, int a_splits, size_t a_ss, s
 extern "C" int odin_heads_linear(const void* a, int a_dtype, int a_splits, long long a_ss, long long a_rs, long long a_hs,
                                  const void* w, int w_dtype, void* out, int out_dtype, long long o_rs, long long o_hs, int T,
                                  int H, int N, int K, const void* gate, int gate_dtype, int gate_splits, long long gate_ss,
-                                 long long gate_rs, void* stream) {
+                                 long long gate_rs, int gate_per_element, void* stream) {
     if (T <= 0) return 0;
     if (a_splits < 1 || (gate != nullptr && gate_splits < 1)) return ODIN_ERR_BAD_ARG;
-    const HeadGate hg{gate, gate_dtype == ODIN_BF16, gate_splits, gate_ss, gate_rs};
+    const HeadGate hg = make_head_gate(gate, gate_dtype, gate_splits, gate_ss, gate_rs, gate_per_element);
     if (H <= 0 || H > 65535 || N <= 0 || K <= 0) return ODIN_ERR_BAD_ARG;
     const size_t smem = (size_t)K * HL_TOK * sizeof(float);
     if (smem > 48 * 1024 || (T + HL_TOK - 1) / HL_TOK > 65535) return ODIN_ERR_UNSUPPORTED;
@@ -290,6 +290,8 @@ extern "C" int odin_heads_linear(const void* a, int a_dtype, int a_splits, long 
     else if (a_dtype == ODIN_F32 && w_dtype == ODIN_F32 && out_dtype == ODIN_F32) GO(float, float, float);
     else if (a_dtype == ODIN_F32 && w_dtype == ODIN_BF16 && out_dtype == ODIN_BF16) GO(float, bf16, bf16);
     else if (a_dtype == ODIN_BF16 && w_dtype == ODIN_F32 && out_dtype == ODIN_BF16) GO(bf16, float, bf16);
+    else if (a_dtype == ODIN_BF16 && w_dtype == ODIN_BF16 && out_dtype == ODIN_F32) GO(bf16, bf16, float);
+    else if (a_dtype == ODIN_BF16 && w_dtype == ODIN_F32 && out_dtype == ODIN_F32) GO(bf16, float, float);
     else return ODIN_ERR_UNSUPPORTED;
 #undef GO
     ODIN_LAUNCH_CHECK();

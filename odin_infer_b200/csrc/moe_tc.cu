@@ -170,7 +170,7 @@ struct GroupedParams {
     int* error;
     // A product per head (tile_expert null): blockIdx.z is the head, which stands in for the expert; row tiles are tiles of
     // tokens, a head's input columns start at head * a_hs of the token's row and its output columns at head * o_hs, and
-    // its outputs are multiplied by the head's gate.
+    // its outputs are multiplied by the head's gate (or by a gate per element).
     int rows;
     long long a_hs, o_hs;
     HeadGate gate;
@@ -308,6 +308,27 @@ moe_grouped_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_const
                     if (per_head) {
 #pragma unroll
                         for (int q = 0; q < 32; ++q) r[q] = __float_as_uint(__uint_as_float(r[q]) * factor);
+                        const int j0g = tile_n * TILE_N + c0;
+                        if (p.gate.per_element && p.gate.p != nullptr && stored && j0g < p.N) {
+                            const int g0 = e * p.N + j0g;
+                            if (p.gate.aligned4 && (p.N & 3) == 0) {
+#pragma unroll
+                                for (int q = 0; q < 32; q += 4) {
+                                    if (j0g + q < p.N) {
+                                        const float4 f = p.gate.sigmoid4_at((int)i, g0 + q);
+                                        r[q] = __float_as_uint(__uint_as_float(r[q]) * f.x);
+                                        r[q + 1] = __float_as_uint(__uint_as_float(r[q + 1]) * f.y);
+                                        r[q + 2] = __float_as_uint(__uint_as_float(r[q + 2]) * f.z);
+                                        r[q + 3] = __float_as_uint(__uint_as_float(r[q + 3]) * f.w);
+                                    }
+                                }
+                            } else {
+#pragma unroll
+                                for (int q = 0; q < 32; ++q)
+                                    if (j0g + q < p.N)
+                                        r[q] = __float_as_uint(__uint_as_float(r[q]) * p.gate.sigmoid_at((int)i, g0 + q));
+                            }
+                        }
                     }
                     if (p.act != 0) {
 #pragma unroll
@@ -497,10 +518,12 @@ extern "C" int odin_moe_grouped(const void* a, long long lda, const void* w, lon
 }
 
 // A product per head for many tokens: out[t, h * o_hs + n] = sigmoid(gate[t, h]) * sum_k a[t, h * a_hs + k] w[h][n][k].
-// a: [T, a_cols] bfloat16 of row stride lda; w: [H][N][K] bfloat16, K a multiple of 64; out: bfloat16 of row stride ldc.
+// (gate_per_element: sigmoid(gate[t, h * N + n]).)  a: [T, a_cols] bfloat16 of row stride lda; w: [H][N][K] bfloat16, K a
+// multiple of 64; out: bfloat16 or 32-bit, of row stride ldc.
 extern "C" int odin_heads_linear_tc(const void* a, long long lda, long long a_hs, int a_cols, const void* w, void* out,
-                                    long long ldc, long long o_hs, int T, int H, int N, int K, const void* gate,
-                                    int gate_dtype, int gate_splits, long long gate_ss, long long gate_rs, void* stream) {
+                                    int out_dtype, long long ldc, long long o_hs, int T, int H, int N, int K,
+                                    const void* gate, int gate_dtype, int gate_splits, long long gate_ss,
+                                    long long gate_rs, int gate_per_element, void* stream) {
     if (T <= 0) return 0;
     if (H <= 0 || H > 65535 || N <= 0 || K <= 0 || (gate != nullptr && gate_splits < 1)) return ODIN_ERR_BAD_ARG;
     if ((lda % 8) || (a_hs % 8) || (K % 64) || (((uintptr_t)a) & 15) || (((uintptr_t)w) & 15) || T > 65535 * BM) return ODIN_ERR_UNSUPPORTED;
@@ -512,7 +535,9 @@ extern "C" int odin_heads_linear_tc(const void* a, long long lda, long long a_hs
     p.out = out; p.ldc = ldc; p.N = N; p.K = K; p.rows_per_expert = N; p.stages = 2;
     p.error = error_flag();
     p.rows = T; p.a_hs = a_hs; p.o_hs = o_hs;
-    p.gate = HeadGate{gate, gate_dtype == ODIN_BF16, gate_splits, gate_ss, gate_rs};
+    p.gate = make_head_gate(gate, gate_dtype, gate_splits, gate_ss, gate_rs, gate_per_element);
+    if (out_dtype == ODIN_F32) return launch_grouped<false, float>(ma, mw, p, (T + BM - 1) / BM, (cudaStream_t)stream, H);
+    if (out_dtype != ODIN_BF16) return ODIN_ERR_UNSUPPORTED;
     return launch_grouped<false, bf16>(ma, mw, p, (T + BM - 1) / BM, (cudaStream_t)stream, H);
 }
 

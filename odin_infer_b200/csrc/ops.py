@@ -75,13 +75,13 @@ def _fn(group: str, name: str):
 
 # ----------------------------------------------------------------------------
 def embed(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, scale: float = 1.0) -> None:
-    """out[t, :] = table[ids[t], :] * scale as 32-bit floats; ids int32 [T]."""
-    T, d = out.shape
+    """out[t, :] = table[ids[t], :] * scale as 32-bit floats; ids int32 [T].  out [copies, T, d]: the same rows in every copy."""
+    T, d = out.shape[-2:]
     assert out.dtype == torch.float32 and ids.dtype == torch.int32 and table.shape[1] == d
     assert table.is_contiguous() and out.is_contiguous()
     _check(_fn("elementwise", "odin_embed")(
         _ptr(table), c_int(dtype_code(table.dtype)), _ptr(ids), _ptr(out), c_int(T), c_int(d),
-        c_int(table.shape[0]), c_float(scale), _stream()), "embed")
+        c_int(table.shape[0]), c_float(scale), c_int(out.shape[0] if out.dim() == 3 else 1), _stream()), "embed")
 
 
 def embed_pair(table: torch.Tensor, pair: torch.Tensor, ids: torch.Tensor, tok_seq: torch.Tensor, seq_start: torch.Tensor,
@@ -91,15 +91,17 @@ def embed_pair(table: torch.Tensor, pair: torch.Tensor, ids: torch.Tensor, tok_s
     token before in the sequence: the row above, or what `state` (int32 [slots, >= 1], any row stride) holds for the
     sequence's slot (token + 1; 0: the sequence starts here, and row `buckets` of `pair` stands in).  A second kernel
     then stores every sequence's last token of this step in `state`.  Rows of sequence -1 become zeros.
-    single_rows: every sequence brings exactly one row; the one kernel then stores the token itself."""
-    T, d = out.shape
+    single_rows: every sequence brings exactly one row; the one kernel then stores the token itself.
+    out [copies, T, d]: the same rows in every copy."""
+    T, d = out.shape[-2:]
     assert out.dtype == torch.float32 and out.is_contiguous() and ids.dtype == torch.int32
     assert table.shape[1] == d and tuple(pair.shape) == (buckets + 1, d) and pair.dtype == table.dtype
     assert table.is_contiguous() and pair.is_contiguous() and state.dtype == torch.int32 and state.stride(1) == 1
     _check(_fn("elementwise", "odin_embed_pair")(
         _ptr(table), _ptr(pair), c_int(dtype_code(table.dtype)), _ptr(ids), _ptr(tok_seq), _ptr(seq_start), _ptr(seq_slots),
         _ptr(state), c_longlong(state.stride(0)), c_int(n_seqs), c_int(buckets), c_longlong(mul_prev), c_longlong(mul_cur),
-        _ptr(out), c_int(T), c_int(d), c_int(table.shape[0]), c_float(scale), c_int(1 if single_rows else 0), _stream()),
+        _ptr(out), c_int(T), c_int(d), c_int(table.shape[0]), c_float(scale), c_int(1 if single_rows else 0),
+        c_int(out.shape[0] if out.dim() == 3 else 1), _stream()),
         "embed_pair", kernels=1 if single_rows else 2)
 
 
@@ -309,12 +311,34 @@ def _vec(w: torch.Tensor | None) -> tuple:
 class Term:
     """One term of a combined update (see `combine_add`): `value` [n, d] or [parts, n, d] partial sums, times `scale`,
     times row_scale[r] (float32 [n]) where given; with norm_weight ([d]) the summed row is first divided by its root mean
-    square (norm_eps inside the root) and multiplied by that weight."""
+    square (norm_eps inside the root) and multiplied by that weight.  bias ([d]): added to the summed row before all that."""
 
     def __init__(self, value: torch.Tensor, scale: float = 1.0, row_scale: torch.Tensor | None = None,
-                 norm_weight: torch.Tensor | None = None, norm_eps: float = 0.0):
+                 norm_weight: torch.Tensor | None = None, norm_eps: float = 0.0, bias: torch.Tensor | None = None):
         self.value, self.scale, self.row_scale = value, float(scale), row_scale
-        self.norm_weight, self.norm_eps = norm_weight, float(norm_eps)
+        self.norm_weight, self.norm_eps, self.bias = norm_weight, float(norm_eps), bias
+
+
+def _term_args(terms: list, rows: int, d: int) -> list:
+    """The kernels' arguments for a list of terms, each of `rows` rows of d elements."""
+    assert len(terms) <= 4
+    n = len(terms)
+    ptrs, dts, nsp, sst, scl = (c_void_p * n)(), (c_int * n)(), (c_int * n)(), (c_longlong * n)(), (c_float * n)()
+    rsc, nws, nwd, nep = (c_void_p * n)(), (c_void_p * n)(), (c_int * n)(), (c_float * n)()
+    bis, bid = (c_void_p * n)(), (c_int * n)()
+    for i, t in enumerate(terms):
+        v = t.value
+        ns, st = _parts(v, rows, d)
+        ptrs[i], dts[i], nsp[i], sst[i], scl[i] = _ptr(v), dtype_code(v.dtype), ns, st, t.scale
+        if t.row_scale is not None:
+            assert t.row_scale.dtype == torch.float32 and t.row_scale.is_contiguous() and t.row_scale.numel() == rows
+        rsc[i] = _ptr(t.row_scale)
+        for w in (t.norm_weight, t.bias):
+            assert w is None or (w.numel() == d and w.is_contiguous())
+        nws[i], nwd[i] = _vec(t.norm_weight)
+        bis[i], bid[i] = _vec(t.bias)
+        nep[i] = t.norm_eps
+    return [c_int(n), ptrs, dts, nsp, sst, scl, rsc, nws, nwd, nep, bis, bid]
 
 
 def combine_add(x: torch.Tensor | None, terms: list, post_weight: torch.Tensor | None = None, post_eps: float = 0.0,
@@ -326,7 +350,6 @@ def combine_add(x: torch.Tensor | None, terms: list, post_weight: torch.Tensor |
     post_center / next_center: the norm is a layer norm (the row's mean is taken off first, the variance is the mean of the
     squared deviations); post_bias / next_bias: added after the weight.  x None: out (float32) = y.  Rows of sequence
     -1 (tok_seq) are skipped.  All sums 32-bit, in an order that the width fixes."""
-    assert len(terms) <= 4
     ref = x if x is not None else out
     d = ref.shape[-1]
     n_all = x.shape[0] if x is not None else out.shape[0]
@@ -337,29 +360,36 @@ def combine_add(x: torch.Tensor | None, terms: list, post_weight: torch.Tensor |
         assert out.is_contiguous() and tuple(out.shape) == (n_rows, d)
     if rows is not None:
         assert rows.dtype == torch.int32
-    n = len(terms)
-    ptrs, dts, nsp, sst, scl = (c_void_p * n)(), (c_int * n)(), (c_int * n)(), (c_longlong * n)(), (c_float * n)()
-    rsc, nws, nwd, nep = (c_void_p * n)(), (c_void_p * n)(), (c_int * n)(), (c_float * n)()
-    for i, t in enumerate(terms):
-        v = t.value
-        ns, st = _parts(v, n_all, d)
-        ptrs[i], dts[i], nsp[i], sst[i], scl[i] = _ptr(v), dtype_code(v.dtype), ns, st, t.scale
-        if t.row_scale is not None:
-            assert t.row_scale.dtype == torch.float32 and t.row_scale.is_contiguous() and t.row_scale.numel() == n_all
-        rsc[i] = _ptr(t.row_scale)
-        if t.norm_weight is not None:
-            assert t.norm_weight.numel() == d and t.norm_weight.is_contiguous()
-        nws[i], nwd[i] = _ptr(t.norm_weight), dtype_code(t.norm_weight.dtype) if t.norm_weight is not None else 0
-        nep[i] = t.norm_eps
     for w in (post_weight, next_weight, post_bias, next_bias):
         assert w is None or (w.numel() == d and w.is_contiguous())
     assert (post_bias is None or post_weight is not None) and (next_bias is None or next_weight is not None)
     _check(_fn("rowwise", "odin_combine_add")(
-        _ptr(x), c_int(n), ptrs, dts, nsp, sst, scl, rsc, nws, nwd, nep, *_vec(post_weight), *_vec(post_bias),
+        _ptr(x), *_term_args(terms, n_all, d), *_vec(post_weight), *_vec(post_bias),
         c_float(post_eps), c_int(1 if post_center else 0), *_vec(next_weight), *_vec(next_bias), c_float(next_eps),
         c_int(1 if next_center else 0), _ptr(out),
         c_int(dtype_code(out.dtype) if out is not None else 0), _ptr(rows), _ptr(tok_seq), c_int(n_rows), c_int(d),
         _stream()), "combine_add")
+
+
+MAX_STREAMS = 16
+
+
+def mix_streams(x: torch.Tensor, terms: list, mix: torch.Tensor | None, add: torch.Tensor | None, read: torch.Tensor,
+                weight: torch.Tensor, eps: float, out: torch.Tensor, rows: torch.Tensor | None = None) -> None:
+    """A residual of s streams, x float32 [s, n, d]: with y the sum of up to four `Term`s, X[j] <- sum_i mix[i, j] X[i] +
+    add[j] y for all streams at once (in place unless `rows` gathers; no terms: the streams stay), then out =
+    weight * u / sqrt(mean(u^2) + eps) with u = sum_j read[j] X[j].  mix [s, s], add and read [s]: float32."""
+    s, n, d = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous() and out.is_contiguous() and weight.numel() == d and weight.is_contiguous()
+    assert tuple(out.shape) == (n if rows is None else rows.numel(), d) and (rows is None or rows.dtype == torch.int32)
+    assert read.dtype == torch.float32 and read.is_contiguous() and read.numel() == s
+    if terms:
+        assert mix.dtype == add.dtype == torch.float32 and mix.is_contiguous() and add.is_contiguous()
+        assert tuple(mix.shape) == (s, s) and add.numel() == s
+    _check(_fn("streams", "odin_mix_streams")(
+        _ptr(x), c_longlong(n * d), c_int(s), c_int(1 if terms else 0), *_term_args(terms, n, d), _ptr(mix if terms else None),
+        _ptr(add if terms else None), _ptr(read), *_vec(weight), c_float(eps), _ptr(out), c_int(dtype_code(out.dtype)),
+        _ptr(rows), c_int(out.shape[0]), c_int(d), _stream()), "mix_streams")
 
 
 def moe_router(h: torch.Tensor, w: torch.Tensor, bias: torch.Tensor | None, top: int, always: int,
@@ -547,7 +577,7 @@ def token_shift(h: torch.Tensor, state: torch.Tensor, mu: torch.Tensor, out: tor
         c_int(T), c_int(d), _stream()), "token_shift")
 
 
-RECURRENCE_MODES = {"bonus": 0, "gated": 1, "fixed": 2, "gla": 3, "ssd": 4}
+RECURRENCE_MODES = {"bonus": 0, "gated": 1, "fixed": 2, "gla": 3, "ssd": 4, "fixed_silu": 5}
 
 
 def linear_recurrence(mode: str, q: torch.Tensor, k: torch.Tensor | None, g: torch.Tensor | None, v: torch.Tensor,
@@ -561,6 +591,7 @@ def linear_recurrence(mode: str, q: torch.Tensor, k: torch.Tensor | None, g: tor
     "bonus": w = exp(-exp(g + c0)); o = (S + diag(c1) k v^T)^T q; S = diag(w) S + k v^T
     "gated": f = c1 + (1 - c1) sigmoid(g + c0); S = diag(f) S + (1 - f) v^T; o = S^T silu(q)
     "fixed": S = c0 S + k v^T; o = S^T q (one constant decay per head, c0: [H]; g and c1 unused)
+    "fixed_silu": as "fixed" with q, k and v through SiLU
     "gla":   w = sigmoid(g + c0)^c1 (as exp(c1 logsigmoid(g + c0))); S = diag(w) S + k v^T; o = S^T (q_scale q)
     "ssd":   per head and token dt = softplus(g[t, head] + c1[head]), w = exp(-exp(c0[head]) dt) (g: [T, H], c0, c1: [H]);
              S = w S + (dt k) v^T; o = S^T q; q and k are [T, (H / heads_per_group) dk]: heads_per_group heads share them
@@ -574,12 +605,12 @@ def linear_recurrence(mode: str, q: torch.Tensor, k: torch.Tensor | None, g: tor
     state from block to block and add each block's incoming state to its tokens' outputs.  The same values up
     to rounding (sums in another order); for long prompts, which one walk per head cannot fill the GPU with."""
     if g is None:
-        assert mode == "fixed"
+        assert mode in ("fixed", "fixed_silu")
         g = q
     for t in (q, g, v, out) + ((k,) if k is not None else ()):
         assert t.dtype == torch.float32 and t.stride(1) == 1
     assert state.dtype == torch.float32 and state.stride(1) == 1 and c0.dtype == c1.dtype
-    per = n_heads if mode in ("fixed", "ssd") else n_heads * dk
+    per = n_heads if mode in ("fixed", "fixed_silu", "ssd") else n_heads * dk
     assert c0.numel() == per and c1.numel() == per
     kk = k if k is not None else q
     width = 0
@@ -650,13 +681,16 @@ def delta_rule(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a: torch.Tenso
 
 def causal_conv(src: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | None, silu: bool, state: torch.Tensor,
                 tok_seq: torch.Tensor, seq_start: torch.Tensor, seq_slots: torch.Tensor, n_seqs: int, out: torch.Tensor,
-                single_rows: bool = False) -> None:
+                single_rows: bool = False, in_bias: torch.Tensor | None = None) -> None:
     """out[t, c] = act(bias[c] + sum_j weight[c, j] src[t - (taps - 1 - j), c]) over each sequence's rows (act: SiLU or
     none); the rows before a step's first one come from `state` (float32 [slots, >= (taps - 1) C], any row stride: the
     sequence's last taps - 1 inputs, oldest first; zeros at its start), into which a second kernel stores the step's last
     inputs.  src: [T, C], a strided view is fine.  single_rows: every sequence brings exactly one row; the one kernel
-    then stores the memory itself."""
+    then stores the memory itself.  in_bias (float32 [C]): added to every input first (the memory holds the sums; what lies
+    before a sequence's start stays zero)."""
     T, C = out.shape
+    if in_bias is not None:
+        assert in_bias.dtype == torch.float32 and in_bias.is_contiguous() and in_bias.numel() == C
     taps = weight.shape[1]
     assert src.stride(1) == 1 and tuple(src.shape) == (T, C) and out.stride(1) == 1
     assert weight.is_contiguous() and weight.shape[0] == C and state.dtype == torch.float32 and state.stride(1) == 1
@@ -668,7 +702,7 @@ def causal_conv(src: torch.Tensor, weight: torch.Tensor, bias: torch.Tensor | No
         _ptr(bias), c_int(dtype_code(bias.dtype) if bias is not None else 0), c_int(taps), c_int(1 if silu else 0),
         _ptr(state), c_longlong(state.stride(0)), _ptr(tok_seq), _ptr(seq_start), _ptr(seq_slots), c_int(n_seqs), _ptr(out),
         c_int(dtype_code(out.dtype)), c_longlong(out.stride(0)), c_int(T), c_int(C), c_int(1 if single_rows else 0),
-        _stream()), "causal_conv", kernels=2 if (taps > 1 and not single_rows) else 1)
+        _ptr(in_bias), _stream()), "causal_conv", kernels=2 if (taps > 1 and not single_rows) else 1)
 
 
 def selective_scan(x: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor | None, B: torch.Tensor, C: torch.Tensor,
@@ -712,10 +746,11 @@ def selective_scan(x: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor | No
 
 
 def skip_gate_norm(o: torch.Tensor, x: torch.Tensor | None, D: torch.Tensor | None, head_dim: int, z: torch.Tensor | None,
-                   weight: torch.Tensor | None, groups: int, eps: float, out: torch.Tensor) -> None:
+                   weight: torch.Tensor | None, groups: int, eps: float, out: torch.Tensor, sigmoid_after: bool = False) -> None:
     """out = weight * grouped_rms((o + D[head] x) * silu(z)): the row of `inner` elements (heads of head_dim) is cut into
     `groups` equal consecutive parts, each divided by its own root mean square.  o float32 [T, inner] contiguous; x float32
-    view; z any view; D [heads] and weight [inner] of one element type; D (with x), z and weight are optional."""
+    view; z any view; D [heads] and weight [inner] of one element type; D (with x), z and weight are optional.  sigmoid_after: z
+    gates the result instead, out = weight * grouped_rms(o + D[head] x) * sigmoid(z)."""
     T, inner = o.shape
     assert o.dtype == torch.float32 and o.is_contiguous() and out.is_contiguous() and tuple(out.shape) == (T, inner)
     if D is not None:
@@ -728,7 +763,53 @@ def skip_gate_norm(o: torch.Tensor, x: torch.Tensor | None, D: torch.Tensor | No
         _ptr(o), _ptr(x if D is not None else None), c_longlong(x.stride(0) if D is not None else 0), _ptr(D),
         c_int(head_dim), _ptr(z), c_int(dtype_code(zd)), c_longlong(z.stride(0) if z is not None else 0), _ptr(weight),
         c_int(dtype_code(wd)), c_int(groups), c_float(eps), _ptr(out), c_int(dtype_code(out.dtype)), c_int(T), c_int(inner),
-        _stream()), "skip_gate_norm")
+        c_int(1 if sigmoid_after else 0), _stream()), "skip_gate_norm")
+
+
+def _gated_unit_args(u, gate_bias, log_decay, y, y_bias, state, out):
+    T, n = u.shape
+    assert u.is_contiguous() and out.is_contiguous() and tuple(out.shape) == (T, n) and out.dtype == u.dtype == y.dtype
+    assert tuple(y.shape) == (T, n) and y.stride(1) == 1 and state.dtype == torch.float32 and state.stride(1) == 1 and state.shape[1] >= n
+    for v, k in ((gate_bias, 2 * n), (log_decay, n), (y_bias, n)):
+        assert v.dtype == torch.float32 and v.is_contiguous() and v.numel() == k
+    return T, n
+
+
+def gated_unit_step(u: torch.Tensor, w: torch.Tensor, gate_bias: torch.Tensor, log_decay: torch.Tensor, y: torch.Tensor,
+                    y_bias: torch.Tensor, state: torch.Tensor, out: torch.Tensor, tok_seq: torch.Tensor,
+                    seq_slots: torch.Tensor) -> None:
+    """One token per sequence of the gated linear unit, its gate products included: with the row u cut into w.shape[0]
+    blocks of m channels and w [blocks, m, 2 m] (input channel before output; r columns, then i columns), gate_bias
+    [blocks, 2 m]:  log a = log_decay * sigmoid(r), S <- a S + sqrt(1 - a^2) sigmoid(i) u, out = S * gelu_tanh(y + y_bias).
+    state: float32 [slots, >= n], any row stride.  Rows of sequence -1 are skipped."""
+    T, n = _gated_unit_args(u, gate_bias, log_decay, y, y_bias, state, out)
+    blocks, m, _ = w.shape
+    assert w.is_contiguous() and blocks * m == n and w.shape[2] == 2 * m
+    _check(_fn("gated_unit", "odin_gated_unit_step")(
+        _ptr(u), c_int(dtype_code(u.dtype)), _ptr(w), c_int(dtype_code(w.dtype)), _ptr(gate_bias), _ptr(log_decay), _ptr(y),
+        c_longlong(y.stride(0)), _ptr(y_bias), _ptr(state), c_longlong(state.stride(0)), _ptr(out), _ptr(tok_seq),
+        _ptr(seq_slots), c_int(T), c_int(n), c_int(blocks), _stream()), "gated_unit_step")
+
+
+def gated_unit_scan(u: torch.Tensor, raw: torch.Tensor, gate_bias: torch.Tensor, log_decay: torch.Tensor, y: torch.Tensor,
+                    y_bias: torch.Tensor, state: torch.Tensor, out: torch.Tensor, seq_start: torch.Tensor,
+                    seq_slots: torch.Tensor, n_seqs: int, max_new: int, block_len: int = 0) -> None:
+    """The same over each sequence's rows in order, the gates' products formed before: raw float32 [T, 2 n], block by block
+    as gate_bias ([blocks, 2 m]) lies.  max_new: the most rows that a sequence brings; its rows are cut into blocks of
+    block_len (0: a choice by max_new) that run side by side, with the state carried from block to block."""
+    T, n = _gated_unit_args(u, gate_bias, log_decay, y, y_bias, state, out)
+    assert raw.dtype == torch.float32 and raw.is_contiguous() and tuple(raw.shape) == (T, 2 * n) and max_new > 0
+    block_len = block_len or (64 if max_new <= 4096 else 256)
+    n_blocks = (max_new + block_len - 1) // block_len
+    s_own = d_own = s_first = None
+    if n_blocks > 1:
+        s_own, d_own = (torch.empty(n_seqs * n_blocks, n, dtype=torch.float32, device=u.device) for _ in range(2))
+        s_first = torch.empty(n_seqs, n, dtype=torch.float32, device=u.device)
+    _check(_fn("gated_unit", "odin_gated_unit_scan")(
+        _ptr(u), c_int(dtype_code(u.dtype)), _ptr(raw), _ptr(gate_bias), _ptr(log_decay), _ptr(y), c_longlong(y.stride(0)),
+        _ptr(y_bias), _ptr(state), c_longlong(state.stride(0)), _ptr(out), _ptr(seq_start), _ptr(seq_slots), c_int(n_seqs),
+        c_int(n), c_int(gate_bias.shape[0]), c_int(block_len), c_int(n_blocks), _ptr(s_own), _ptr(d_own), _ptr(s_first),
+        _stream()), "gated_unit_scan", kernels=2 if n_blocks > 1 else 1)
 
 
 def head_unit_scale(o: torch.Tensor, weight: torch.Tensor | None, per_head_weight: bool, gate: torch.Tensor | None,
@@ -793,22 +874,23 @@ def heads_linear(a: torch.Tensor, a_head_stride: int, w: torch.Tensor, out: torc
     """A product per head: out[t, h * out_head_stride + n] = sum_k a[t, h * a_head_stride + k] * w[h, k, n] for
     w [H, K, N] (input channel before output channel); a and out may be views with any row stride, a also float32 partial
     sums [parts, T, ...] of a split product.  gate ([T, H], a view or partial sums): head h's outputs are multiplied by
-    sigmoid(gate[t, h])."""
+    sigmoid(gate[t, h]); a gate of [T, H N] has a number per output, sigmoid(gate[t, h * N + n])."""
     H, K, N = w.shape
     T = a.shape[-2]
     assert w.is_contiguous() and a.stride(-1) == 1 and out.stride(1) == 1 and out.shape[0] == T
     assert a.shape[-1] >= (H - 1) * a_head_stride + K and out.shape[1] >= (H - 1) * out_head_stride + N
     a_split, a_ss, a_rs = _parts_view(a)
-    g_split, g_ss, g_rs = (1, 0, 0)
+    g_split, g_ss, g_rs, per_element = (1, 0, 0, False)
     if gate is not None:
-        assert tuple(gate.shape[-2:]) == (T, H)
+        per_element = gate.shape[-1] != H
+        assert tuple(gate.shape[-2:]) == (T, H * N if per_element else H)
         g_split, g_ss, g_rs = _parts_view(gate)
     _check(_fn("latent", "odin_heads_linear")(
         _ptr(a), c_int(dtype_code(a.dtype)), c_int(a_split), c_longlong(a_ss), c_longlong(a_rs), c_longlong(a_head_stride),
         _ptr(w), c_int(dtype_code(w.dtype)), _ptr(out), c_int(dtype_code(out.dtype)), c_longlong(out.stride(0)),
         c_longlong(out_head_stride), c_int(T), c_int(H), c_int(N), c_int(K), _ptr(gate),
         c_int(dtype_code(gate.dtype) if gate is not None else 0), c_int(g_split), c_longlong(g_ss), c_longlong(g_rs),
-        _stream()), "heads_linear")
+        c_int(1 if per_element else 0), _stream()), "heads_linear")
 
 
 def heads_linear_tc_supported(a: torch.Tensor, a_head_stride: int, w: torch.Tensor) -> bool:
@@ -821,22 +903,23 @@ def heads_linear_tc_supported(a: torch.Tensor, a_head_stride: int, w: torch.Tens
 def heads_linear_tc(a: torch.Tensor, a_head_stride: int, w: torch.Tensor, out: torch.Tensor, out_head_stride: int,
                     gate: torch.Tensor | None = None) -> None:
     """`heads_linear` on the tcgen05 tensor cores, for many tokens: w is [H, N, K] (output channel before input channel),
-    a and out bfloat16."""
+    a bfloat16, out bfloat16 or float32."""
     H, N, K = w.shape
     T = a.shape[0]
     if not heads_linear_tc_supported(a, a_head_stride, w):
         raise KernelError("heads_linear_tc: bfloat16 rows of whole 16 bytes and K a multiple of 64")
-    assert out.dtype == torch.bfloat16 and out.stride(1) == 1 and out.shape[0] == T
+    assert out.stride(1) == 1 and out.shape[0] == T
     assert a.shape[1] >= (H - 1) * a_head_stride + K and out.shape[1] >= (H - 1) * out_head_stride + N
-    g_split, g_ss, g_rs = (1, 0, 0)
+    g_split, g_ss, g_rs, per_element = (1, 0, 0, False)
     if gate is not None:
-        assert tuple(gate.shape[-2:]) == (T, H)
+        per_element = gate.shape[-1] != H
+        assert tuple(gate.shape[-2:]) == (T, H * N if per_element else H)
         g_split, g_ss, g_rs = _parts_view(gate)
     _check(_fn("moe_tc", "odin_heads_linear_tc")(
         _ptr(a), c_longlong(a.stride(0)), c_longlong(a_head_stride), c_int(a.shape[1]), _ptr(w), _ptr(out),
-        c_longlong(out.stride(0)), c_longlong(out_head_stride), c_int(T), c_int(H), c_int(N), c_int(K), _ptr(gate),
+        c_int(dtype_code(out.dtype)), c_longlong(out.stride(0)), c_longlong(out_head_stride), c_int(T), c_int(H), c_int(N), c_int(K), _ptr(gate),
         c_int(dtype_code(gate.dtype) if gate is not None else 0), c_int(g_split), c_longlong(g_ss), c_longlong(g_rs),
-        _stream()), "heads_linear_tc")
+        c_int(1 if per_element else 0), _stream()), "heads_linear_tc")
 
 
 def rope_heads(src: torch.Tensor, src_head_stride: int, dst: torch.Tensor, dst_head_stride: int, n_heads: int, width: int,
@@ -1009,7 +1092,8 @@ def head_prep(qkv: torch.Tensor, n_q: int, n_kv: int, head_dim: int, q_norm: tor
               k_cache: torch.Tensor | None, v_cache: torch.Tensor | None, write_kv: bool = True,
               q_out: torch.Tensor | None = None, bias: torch.Tensor | None = None, unit_norm_after: bool = False,
               v_head_dim: int | None = None, whole_norm: bool = False, pairs: bool = False,
-              v_first: torch.Tensor | None = None, v_lambda: float = 0.0, v_keep: torch.Tensor | None = None) -> torch.Tensor:
+              v_first: torch.Tensor | None = None, v_lambda: float = 0.0, v_keep: torch.Tensor | None = None,
+              values_are_keys: bool = False) -> torch.Tensor:
     """Per-head RMSNorm and rotation of q and k, and the cache write of k and v.
 
     bias: one value per column of the projection, added first.  unit_norm_after: instead of the
@@ -1024,7 +1108,8 @@ def head_prep(qkv: torch.Tensor, n_q: int, n_kv: int, head_dim: int, q_norm: tor
     product (added first).  q goes to q_out ([T, n_q head_dim], of the cache's type); without
     q_out it is written back into qkv (one part only).  Returns the tensor that holds q."""
     vd = head_dim if v_head_dim is None else v_head_dim
-    width = (n_q + n_kv) * head_dim + n_kv * vd
+    width = (n_q + n_kv) * head_dim + (0 if values_are_keys else n_kv * vd)
+    assert not values_are_keys or (vd == head_dim and v_first is None and v_keep is None)
     if qkv.dim() == 3:
         n_split, T = qkv.shape[0], qkv.shape[1]
         assert qkv.is_contiguous() and qkv.shape[2] >= width   # further columns (a gate's) are left alone
@@ -1065,8 +1150,8 @@ def head_prep(qkv: torch.Tensor, n_q: int, n_kv: int, head_dim: int, q_norm: tor
         c_float(eps),
         _ptr(cos), _ptr(sin), c_int(rotary_dim), c_int(cos.shape[0]), _ptr(tok_pos), _ptr(tok_seq),
         _ptr(block_table), c_int(block_table.stride(0)), _ptr(k_cache), _ptr(v_cache), c_int(PAGE),
-        c_int(1 if write_kv else 0), c_int(1 if pairs else 0), _ptr(v_first), _ptr(v_keep), c_float(v_lambda), _stream()),
-        "head_prep")
+        c_int(1 if write_kv else 0), c_int(1 if pairs else 0), _ptr(v_first), _ptr(v_keep), c_float(v_lambda),
+        c_int(1 if values_are_keys else 0), _stream()), "head_prep")
     return q_out
 
 

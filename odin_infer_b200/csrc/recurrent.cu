@@ -81,6 +81,7 @@ extern "C" int odin_token_shift(const void* h, int dtype, const float* state, lo
 #define REC_GLA 3     // w = sigmoid(raw + c0)^c1 = exp(c1 logsigmoid(raw + c0)); S = diag(w) S + k v^T; o = S^T (q_scale q)
 #define REC_SSD 4     // per head and token one step dt = softplus(raw[head] + c1[head]) and one decay w = exp(-exp(c0[head]) dt);
                       // S = w S + (dt k) v^T; o = S^T q; q and k belong to the head's group (heads_per_group heads share them)
+#define REC_FIXED_SILU 5  // as REC_FIXED with q, k and v through SiLU
 // One CTA per (sequence, head) walks the sequence's tokens in order.  Column j of S belongs to REC_SPLIT lanes of
 // one warp (lane = part * 8 + j % 8), each holding SL consecutive key channels of it in registers; a token costs
 // each thread SL multiply-adds for the output and SL for the state, and the column's output is the sum of its
@@ -98,7 +99,8 @@ linear_recurrence_kernel(RecParams p) {
     constexpr int NK = SL * REC_SPLIT;             // key channels the registers hold (dk <= NK)
     constexpr int TOK = NK > 128 ? 8 : 16;
     constexpr bool BONUS_IN_REGS = SL <= 32;
-    constexpr bool UNI = MODE == REC_FIXED || MODE == REC_SSD;   // one decay for the whole head: a register, no row of shared memory
+    constexpr bool FIXED = MODE == REC_FIXED || MODE == REC_FIXED_SILU;
+    constexpr bool UNI = FIXED || MODE == REC_SSD;   // one decay for the whole head: a register, no row of shared memory
     __shared__ float s_wt[TOK], s_dt[TOK];         // REC_SSD: the token's decay and step, formed once per token
     // A warp's four parts read their channels at the same moment, SL floats apart: every part's channels sit four floats
     // further on than the part before, so that the four 16-byte reads fall into different banks (SL = 32: banks 0, 4, 8, 12
@@ -125,7 +127,7 @@ linear_recurrence_kernel(RecParams p) {
     const bool owns = j < p.dv;
     const int i0 = part * SL;
     float S[SL], ub[BONUS_IN_REGS ? SL : 1], D[(BLOCKS && !UNI) ? SL : 1];
-    const float wuni = MODE == REC_FIXED ? p.c0.at(head) : 0.f;
+    const float wuni = FIXED ? p.c0.at(head) : 0.f;
     float* st = BLOCKS ? p.s_loc + ((size_t)blockIdx.x * p.H + head) * dk * p.dv + j
                        : p.state + (size_t)slot * p.state_stride + (size_t)head * dk * p.dv + j;
 #pragma unroll
@@ -153,7 +155,7 @@ linear_recurrence_kernel(RecParams p) {
                     const size_t r = (size_t)(t0 + u);
                     rq[f] = p.q[r * p.q_stride + qc + i];
                     if (MODE == REC_SSD) rg[f] = p.g[r * p.g_stride + head];
-                    else if (MODE != REC_FIXED) rg[f] = p.g[r * p.g_stride + hc + i];
+                    else if (!FIXED) rg[f] = p.g[r * p.g_stride + hc + i];
                     if (MODE != REC_GATED) rk[f] = p.k[r * p.k_stride + qc + i];
                 }
             }
@@ -178,6 +180,9 @@ linear_recurrence_kernel(RecParams p) {
                     } else if (MODE == REC_FIXED) {
                         qv = rq[f];
                         kv = rk[f];
+                    } else if (MODE == REC_FIXED_SILU) {
+                        qv = rq[f] / (1.0f + expf(-rq[f]));
+                        kv = rk[f] / (1.0f + expf(-rk[f]));
                     } else if (MODE == REC_GLA) {
                         const float z = rg[f] + p.c0.at(hc + i);
                         const float logsig = fminf(z, 0.f) - log1pf(expf(-fabsf(z)));
@@ -205,7 +210,8 @@ linear_recurrence_kernel(RecParams p) {
                 sq[u][ip] = qv; sk[u][ip] = kv;
                 if (!UNI) sw[u][ip] = wv;
             }
-            if (e < nt * ccols) sv[e / ccols][e % ccols] = rv[f];
+            if (e < nt * ccols)
+                sv[e / ccols][e % ccols] = MODE == REC_FIXED_SILU ? rv[f] / (1.0f + expf(-rv[f])) : rv[f];
         }
     };
 
@@ -326,7 +332,7 @@ extern "C" int odin_linear_recurrence(int mode, const float* q, long long q_stri
                                             (long long)n_seqs * n_blocks > 2147483647LL)))
         return ODIN_ERR_BAD_ARG;
     if (H <= 0 || dk <= 0 || dk > REC_MAX_DK || dv <= 0 || dv > 256 || H > 65535) return ODIN_ERR_UNSUPPORTED;
-    if (mode < REC_BONUS || mode > REC_SSD) return ODIN_ERR_BAD_ARG;
+    if (mode < REC_BONUS || mode > REC_FIXED_SILU) return ODIN_ERR_BAD_ARG;
     if (mode == REC_SSD && (heads_per_group <= 0 || H % heads_per_group != 0)) return ODIN_ERR_BAD_ARG;
     RecParams p;
     p.q = q; p.q_stride = q_stride; p.k = k; p.k_stride = k_stride; p.g = g; p.g_stride = g_stride;
@@ -357,6 +363,8 @@ extern "C" int odin_linear_recurrence(int mode, const float* q, long long q_stri
         else if (mode == REC_BONUS) odin_launch(linear_recurrence_kernel<SL, REC_BONUS, false>, grid, dim3(threads), 0, s, p);     \
         else if (mode == REC_FIXED && blocks) odin_launch(linear_recurrence_kernel<SL, REC_FIXED, true>, grid, dim3(threads), 0, s, p);  \
         else if (mode == REC_FIXED) odin_launch(linear_recurrence_kernel<SL, REC_FIXED, false>, grid, dim3(threads), 0, s, p);     \
+        else if (mode == REC_FIXED_SILU && blocks) odin_launch(linear_recurrence_kernel<SL, REC_FIXED_SILU, true>, grid, dim3(threads), 0, s, p);  \
+        else if (mode == REC_FIXED_SILU) odin_launch(linear_recurrence_kernel<SL, REC_FIXED_SILU, false>, grid, dim3(threads), 0, s, p);     \
         else if (mode == REC_GLA && blocks) odin_launch(linear_recurrence_kernel<SL, REC_GLA, true>, grid, dim3(threads), 0, s, p);  \
         else if (mode == REC_GLA) odin_launch(linear_recurrence_kernel<SL, REC_GLA, false>, grid, dim3(threads), 0, s, p);     \
         else if (mode == REC_SSD && blocks) odin_launch(linear_recurrence_kernel<SL, REC_SSD, true>, grid, dim3(threads), 0, s, p);  \

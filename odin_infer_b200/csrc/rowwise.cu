@@ -9,7 +9,7 @@
 //     embedding).
 // All arithmetic is 32-bit; a row's sums run in an order fixed by the block size alone, so a
 // row's result does not depend on the other rows of the launch.
-#include "common.cuh"
+#include "combine_terms.cuh"
 
 #define ROW_THREADS 256
 
@@ -557,18 +557,12 @@ extern "C" int odin_softcap(float* z, long long stride, int rows, int n, float c
 
 
 // ------------------------------------------------------------ several terms into one update, normed, added, normed again
-// y = sum_i scale_i * rowscale_i[r] * f_i(sum of term i's parts), f_i the identity or w_i * v / rms(v) over the row;
+// y = sum_i scale_i * rowscale_i[r] * f_i(sum of term i's parts + its bias), f_i the identity or w_i * v / rms(v) over the row;
 // then x[r] += post_w * y / rms(y) (post_w null: x[r] += y), and out = next_w * x[r] / rms(x[r]) (next_w null: out = x[r]
 // converted, or no output at all).  Either of these two norms may be a layer norm (`center`): the row's mean is taken off
 // first, the variance is the mean of the squared deviations, and a bias may follow the weight.
 // Without x the sum itself goes to out as 32-bit values.  rows: gather these rows (x is then left as it is).
 // One CTA per row; every sum runs in an order that the width and the block size fix.
-#define COMBINE_MAX_TERMS 4
-struct CombineTerm {
-    const void* p; int is_bf16; int n_split; long long split_stride;
-    float scale; const float* row_scale; VecRef norm_w; float norm_eps;
-};
-struct CombineArgs { CombineTerm t[COMBINE_MAX_TERMS]; int n; };
 struct CombineNorm { VecRef w, b; float eps; int center; };   // w null: no norm
 
 template <typename TO, bool VEC>
@@ -612,6 +606,11 @@ combine_add_kernel(float* __restrict__ x, CombineArgs a, CombineNorm post, Combi
             for (int e = 0; e < W; ++e) v[e] = 0.f;
             for (int sp = 0; sp < tm.n_split; ++sp) {
                 load(tm, (size_t)sp * tm.split_stride + (size_t)r * d + j, u);
+#pragma unroll
+                for (int e = 0; e < W; ++e) v[e] += u[e];
+            }
+            if (tm.bias.p != nullptr) {
+                weights(tm.bias, j, u);
 #pragma unroll
                 for (int e = 0; e < W; ++e) v[e] += u[e];
             }
@@ -806,8 +805,8 @@ combine_one_kernel(float* __restrict__ x, const TD* __restrict__ delta, int n_sp
 extern "C" int odin_combine_add(float* x, int n_terms, const void* const* ptrs, const int* dtypes, const int* n_splits,
                                 const long long* split_strides, const float* scales, const float* const* row_scales,
                                 const void* const* norm_ws, const int* norm_w_dtypes, const float* norm_eps,
-                                const void* post_w, int post_w_dtype, const void* post_b, int post_b_dtype, float post_eps,
-                                int post_center, const void* next_w, int next_w_dtype, const void* next_b, int next_b_dtype,
+                                const void* const* biases, const int* bias_dtypes, const void* post_w, int post_w_dtype,
+                                const void* post_b, int post_b_dtype, float post_eps, int post_center, const void* next_w, int next_w_dtype, const void* next_b, int next_b_dtype,
                                 float next_eps, int next_center, void* out, int out_dtype, const int* rows,
                                 const int* tok_seq, int n_rows, int d, void* stream) {
     if (n_rows <= 0) return 0;
@@ -817,21 +816,15 @@ extern "C" int odin_combine_add(float* x, int n_terms, const void* const* ptrs, 
     const size_t smem = (size_t)2 * d * sizeof(float);
     if (smem > 200 * 1024) return ODIN_ERR_UNSUPPORTED;
     CombineArgs a;
-    a.n = n_terms;
     uintptr_t all_bits = 0;
-    for (int i = 0; i < n_terms; ++i) {
-        if (dtypes[i] != ODIN_BF16 && dtypes[i] != ODIN_F32) return ODIN_ERR_UNSUPPORTED;
-        a.t[i].p = ptrs[i]; a.t[i].is_bf16 = dtypes[i] == ODIN_BF16; a.t[i].n_split = n_splits[i];
-        a.t[i].split_stride = split_strides[i]; a.t[i].scale = scales[i]; a.t[i].row_scale = row_scales[i];
-        a.t[i].norm_w = VecRef{norm_ws[i], norm_w_dtypes[i] == ODIN_BF16}; a.t[i].norm_eps = norm_eps[i];
-        all_bits |= (uintptr_t)ptrs[i] | (uintptr_t)norm_ws[i] | (uintptr_t)(split_strides[i] * 4);
-    }
+    if (const int rc = fill_combine_args(a, all_bits, n_terms, ptrs, dtypes, n_splits, split_strides, scales, row_scales, norm_ws,
+                                         norm_w_dtypes, norm_eps, biases, bias_dtypes)) return rc;
     all_bits |= (uintptr_t)x | (uintptr_t)out | (uintptr_t)post_w | (uintptr_t)next_w | (uintptr_t)post_b | (uintptr_t)next_b;
     const bool vec = (d % 4 == 0) && (all_bits % 16 == 0);
     cudaStream_t s = (cudaStream_t)stream;
     const CombineNorm post{VecRef{post_w, post_w_dtype == ODIN_BF16}, VecRef{post_b, post_b_dtype == ODIN_BF16}, post_eps, post_center};
     const CombineNorm next{VecRef{next_w, next_w_dtype == ODIN_BF16}, VecRef{next_b, next_b_dtype == ODIN_BF16}, next_eps, next_center};
-    if (vec && x != nullptr && n_terms == 1 && norm_ws[0] == nullptr && row_scales[0] == nullptr && d <= 4 * 1024) {
+    if (vec && x != nullptr && n_terms == 1 && norm_ws[0] == nullptr && row_scales[0] == nullptr && biases[0] == nullptr && d <= 4 * 1024) {
         const int nv = d <= 1024 ? 1 : d <= 2048 ? 2 : 4;
 #define ONE(TD, TO, NV)                                                                                              \
     odin_launch(combine_one_kernel<TD, TO, NV>, dim3(n_rows), dim3(ROW_THREADS), 0, s, x, (const TD*)ptrs[0],         \

@@ -1,6 +1,6 @@
 // State-space mixers: what stands around and inside a selective scan.
 //
-//   * causal convolution per channel over a sequence's rows, with a bias and an optional SiLU; the rows before a
+//   * causal convolution per channel over a sequence's rows, with a bias, an optional bias on its inputs and an optional SiLU; the rows before a
 //     step's first one come from the sequence's state (its last taps - 1 inputs, zeros at a sequence's start), and a
 //     second kernel stores the step's last inputs there;
 //   * the selective scan with one state row per channel:
@@ -27,7 +27,7 @@ __global__ void __launch_bounds__(256)
 causal_conv_kernel(const TI* __restrict__ in, size_t in_stride, VecRef w, VecRef bias, int taps, int silu,
                    float* __restrict__ state, size_t state_stride, const int* __restrict__ tok_seq,
                    const int* __restrict__ seq_start, const int* __restrict__ seq_slots, TO* __restrict__ out,
-                   size_t out_stride, int C, int store) {
+                   size_t out_stride, int C, int store, const float* __restrict__ in_bias) {
     pdl_trigger();
     const int t = blockIdx.x;
     const int c = blockIdx.y * blockDim.x + threadIdx.x;
@@ -37,10 +37,11 @@ causal_conv_kernel(const TI* __restrict__ in, size_t in_stride, VecRef w, VecRef
     pdl_wait();
     if (seq < 0 || c >= C) return;
     float acc = bias.p != nullptr ? bias.at(c) : 0.f;
+    const float ib = in_bias != nullptr ? in_bias[c] : 0.f;   // the memory holds inputs with their bias
     for (int j = 0; j < taps; ++j) {
         const int r = t - (taps - 1 - j);
         float v;
-        if (r >= first) v = to_f32(in[(size_t)r * in_stride + c]);
+        if (r >= first) v = to_f32(in[(size_t)r * in_stride + c]) + ib;
         else v = state[(size_t)slot * state_stride + (size_t)(taps - 1 - (first - r)) * C + c];
         acc = fmaf(w.at(c * taps + j), v, acc);
     }
@@ -48,7 +49,7 @@ causal_conv_kernel(const TI* __restrict__ in, size_t in_stride, VecRef w, VecRef
     if (store && taps > 1) {   // t == first: the memory moves up by one row and takes this row's input
         float* st = state + (size_t)slot * state_stride + c;
         for (int k = 0; k + 2 < taps; ++k) st[(size_t)k * C] = st[(size_t)(k + 1) * C];
-        st[(size_t)(taps - 2) * C] = to_f32(in[(size_t)t * in_stride + c]);
+        st[(size_t)(taps - 2) * C] = to_f32(in[(size_t)t * in_stride + c]) + ib;
     }
 }
 
@@ -61,13 +62,14 @@ __global__ void __launch_bounds__(256)
 causal_conv4_kernel(const TI* __restrict__ in, size_t in_stride, VecRef w, VecRef bias, int taps, int silu,
                     const float* __restrict__ state, size_t state_stride, const int* __restrict__ tok_seq,
                     const int* __restrict__ seq_start, const int* __restrict__ seq_slots, TO* __restrict__ out,
-                    size_t out_stride, int C, int T) {
+                    size_t out_stride, int C, int T, const float* __restrict__ in_bias) {
     pdl_trigger();
     const int t0 = blockIdx.x * CONV_TOK, t1 = min(T, t0 + CONV_TOK);
     const int c = blockIdx.y * blockDim.x + threadIdx.x;
     float wv[4] = {0.f, 0.f, 0.f, 0.f};   // wv[3] meets the current row, wv[3 - m] the row m before
-    float b = 0.f;
+    float b = 0.f, ib = 0.f;
     if (c < C) {
+        if (in_bias != nullptr) ib = in_bias[c];
         for (int j = 0; j < taps; ++j) wv[4 - taps + j] = w.at(c * taps + j);
         if (bias.p != nullptr) b = bias.at(c);
     }
@@ -86,14 +88,14 @@ causal_conv4_kernel(const TI* __restrict__ in, size_t in_stride, VecRef w, VecRe
                 float v = 0.f;
                 if (m < taps) {
                     const int r = t - m;
-                    v = r >= first ? to_f32(in[(size_t)r * in_stride + c])
+                    v = r >= first ? to_f32(in[(size_t)r * in_stride + c]) + ib
                                    : state[(size_t)slot * state_stride + (size_t)(taps - 1 - (first - r)) * C + c];
                 }
                 win[m - 1] = v;
             }
             have = seq;
         }
-        const float cur = to_f32(in[(size_t)t * in_stride + c]);
+        const float cur = to_f32(in[(size_t)t * in_stride + c]) + ib;
         float acc = b;
         if (taps > 3) acc = fmaf(wv[0], win[2], acc);
         if (taps > 2) acc = fmaf(wv[1], win[1], acc);
@@ -108,7 +110,8 @@ causal_conv4_kernel(const TI* __restrict__ in, size_t in_stride, VecRef w, VecRe
 template <typename TI>
 __global__ void __launch_bounds__(256)
 conv_state_kernel(const TI* __restrict__ in, size_t in_stride, int taps, float* __restrict__ state, size_t state_stride,
-                  const int* __restrict__ seq_start, const int* __restrict__ seq_slots, int C) {
+                  const int* __restrict__ seq_start, const int* __restrict__ seq_slots, int C,
+                  const float* __restrict__ in_bias) {
     pdl_trigger();
     const int b = blockIdx.x;
     const int c = blockIdx.y * blockDim.x + threadIdx.x;
@@ -117,16 +120,18 @@ conv_state_kernel(const TI* __restrict__ in, size_t in_stride, int taps, float* 
     if (n_new <= 0 || c >= C) return;
     float* st = state + (size_t)slot * state_stride + c;
     const int keep = taps - 1;
+    const float ib = in_bias != nullptr ? in_bias[c] : 0.f;
     for (int k = 0; k < keep; ++k) {   // ascending: an old value is read before its place is written
         const int p = n_new + k;       // place in (old state ++ new rows)
-        st[(size_t)k * C] = p < keep ? st[(size_t)p * C] : to_f32(in[(size_t)(first + p - keep) * in_stride + c]);
+        st[(size_t)k * C] = p < keep ? st[(size_t)p * C] : to_f32(in[(size_t)(first + p - keep) * in_stride + c]) + ib;
     }
 }
 
 extern "C" int odin_causal_conv(const void* in, int in_dtype, long long in_stride, const void* w, int w_dtype,
                                 const void* bias, int bias_dtype, int taps, int silu, float* state, long long state_stride,
                                 const int* tok_seq, const int* seq_start, const int* seq_slots, int n_seqs, void* out,
-                                int out_dtype, long long out_stride, int T, int C, int single_rows, void* stream) {
+                                int out_dtype, long long out_stride, int T, int C, int single_rows, const float* in_bias,
+                                void* stream) {
     if (T <= 0) return 0;
     if (C <= 0 || taps < 1 || taps > 64 || n_seqs <= 0) return ODIN_ERR_BAD_ARG;
     cudaStream_t s = (cudaStream_t)stream;
@@ -140,11 +145,11 @@ extern "C" int odin_causal_conv(const void* in, int in_dtype, long long in_strid
         if (taps <= 4 && T > 64 && !single_rows)                                                                     \
             odin_launch(causal_conv4_kernel<TI, TO>, grid4, dim3(threads), 0, s, (const TI*)in, (size_t)in_stride, wv, bv, \
                         taps, silu, (const float*)state, (size_t)state_stride, tok_seq, seq_start, seq_slots, (TO*)out, \
-                        (size_t)out_stride, C, T);                                                                   \
+                        (size_t)out_stride, C, T, in_bias);                                                          \
         else                                                                                                         \
             odin_launch(causal_conv_kernel<TI, TO>, grid, dim3(threads), 0, s, (const TI*)in, (size_t)in_stride, wv, bv, \
                         taps, silu, state, (size_t)state_stride, tok_seq, seq_start, seq_slots, (TO*)out,           \
-                        (size_t)out_stride, C, single_rows);                                                         \
+                        (size_t)out_stride, C, single_rows, in_bias);                                                \
     } while (0)
     if (in_dtype == ODIN_BF16 && out_dtype == ODIN_BF16) GO(bf16, bf16);
     else if (in_dtype == ODIN_BF16 && out_dtype == ODIN_F32) GO(bf16, float);
@@ -157,10 +162,10 @@ extern "C" int odin_causal_conv(const void* in, int in_dtype, long long in_strid
         dim3 g2(n_seqs, grid.y);
         if (in_dtype == ODIN_BF16)
             odin_launch(conv_state_kernel<bf16>, g2, dim3(threads), 0, s, (const bf16*)in, (size_t)in_stride, taps, state,
-                        (size_t)state_stride, seq_start, seq_slots, C);
+                        (size_t)state_stride, seq_start, seq_slots, C, in_bias);
         else
             odin_launch(conv_state_kernel<float>, g2, dim3(threads), 0, s, (const float*)in, (size_t)in_stride, taps, state,
-                        (size_t)state_stride, seq_start, seq_slots, C);
+                        (size_t)state_stride, seq_start, seq_slots, C, in_bias);
         ODIN_LAUNCH_CHECK();
     }
     return 0;
@@ -435,11 +440,12 @@ extern "C" int odin_selective_scan(const void* x, int x_dtype, long long x_strid
 // ------------------------------------------------------------ skip, gate and grouped norm after a recurrence over heads
 // y[t, h, j] = (o[t, h, j] + D[h] x[t, h, j]) * silu(z[t, h, j]); the row is cut into `groups` equal consecutive parts and
 // every part is divided by its own root mean square; out = y * w.  One CTA per (token, part); D, z and w are optional.
+// sig_after: z gates the result instead, out = y * w * sigmoid(z), and does not enter the norm.
 template <typename TZ, typename TO>
 __global__ void __launch_bounds__(256)
 skip_gate_norm_kernel(const float* __restrict__ o, const float* __restrict__ x, size_t x_stride, VecRef D, int P,
                       const TZ* __restrict__ z, size_t z_stride, VecRef w, int groups, float eps, TO* __restrict__ out,
-                      int inner) {
+                      int inner, int sig_after) {
     extern __shared__ float row[];   // one part of the row
     __shared__ float red[32];
     pdl_trigger();
@@ -451,7 +457,7 @@ skip_gate_norm_kernel(const float* __restrict__ o, const float* __restrict__ x, 
         const int j = j0 + i;
         float y = o[(size_t)t * inner + j];
         if (D.p != nullptr) y = fmaf(D.at(j / P), x[(size_t)t * x_stride + j], y);
-        if (z != nullptr) y *= ss_silu(to_f32(z[(size_t)t * z_stride + j]));
+        if (z != nullptr && !sig_after) y *= ss_silu(to_f32(z[(size_t)t * z_stride + j]));
         row[i] = y;
         ss += y * y;
     }
@@ -459,13 +465,16 @@ skip_gate_norm_kernel(const float* __restrict__ o, const float* __restrict__ x, 
     ss /= (float)gsz;
     ss += eps;
     const float rs = 1.0f / sqrtf(ss);
-    for (int i = threadIdx.x; i < gsz; i += blockDim.x)
-        out[(size_t)t * inner + j0 + i] = from_f32<TO>(w.p != nullptr ? w.at(j0 + i) * (rs * row[i]) : rs * row[i]);
+    for (int i = threadIdx.x; i < gsz; i += blockDim.x) {
+        float y = w.p != nullptr ? w.at(j0 + i) * (rs * row[i]) : rs * row[i];
+        if (z != nullptr && sig_after) y /= 1.0f + expf(-to_f32(z[(size_t)t * z_stride + j0 + i]));
+        out[(size_t)t * inner + j0 + i] = from_f32<TO>(y);
+    }
 }
 
 extern "C" int odin_skip_gate_norm(const float* o, const float* x, long long x_stride, const void* D, int P, const void* z,
                                    int z_dtype, long long z_stride, const void* w, int w_dtype, int groups, float eps,
-                                   void* out, int out_dtype, int T, int inner, void* stream) {
+                                   void* out, int out_dtype, int T, int inner, int sig_after, void* stream) {
     if (T <= 0) return 0;
     if (inner <= 0 || groups < 1 || inner % groups != 0 || P <= 0) return ODIN_ERR_BAD_ARG;
     const size_t smem = (size_t)(inner / groups) * sizeof(float);
@@ -480,7 +489,7 @@ extern "C" int odin_skip_gate_norm(const float* o, const float* x, long long x_s
             if (e != cudaSuccess) return (int)e;                                                                        \
         }                                                                                                               \
         odin_launch(skip_gate_norm_kernel<TZ, TO>, dim3(T, groups), dim3(threads), smem, s, o, x, (size_t)x_stride, Dv, P, (const TZ*)z, \
-                    (size_t)z_stride, wv, groups, eps, (TO*)out, inner);                                                \
+                    (size_t)z_stride, wv, groups, eps, (TO*)out, inner, sig_after);                                     \
     } while (0)
     if (z_dtype == ODIN_BF16 && out_dtype == ODIN_BF16) GO(bf16, bf16);
     else if (z_dtype == ODIN_F32 && out_dtype == ODIN_F32) GO(float, float);

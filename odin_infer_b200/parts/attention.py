@@ -35,6 +35,9 @@ class GQAttention(Mixer):
     value_mix = {"key": str, "lambda": name of a scalar tensor or None}: values are mixed with those of an earlier layer of
     the same step.  Without a "lambda" this mixer's own values are kept under `key` for the layers after it; with one, what
     it attends over (and caches) is (1 - lambda) v + lambda v_kept.
+    values_are_keys: there is no value projection; the values are the keys as projected (bias included), before their norm
+    and rotation.  sink_logit: a fixed number in place of a learned `sink`, the same for all heads (0: one is added to the
+    softmax's denominator).
     """
 
     graph_safe = True
@@ -44,7 +47,8 @@ class GQAttention(Mixer):
                  position_encoding: str | None = None, qk_norm=True, eps: float = 1e-6,
                  window: int = 0, kv_shared: bool = False, chunk: int = 0, biases: dict | None = None,
                  scale: float = 0.0, softcap: float = 0.0, v_head_dim: int = 0, sink: str | None = None,
-                 gate: str | None = None, gate_per_head: bool = False, value_mix: dict | None = None):
+                 gate: str | None = None, gate_per_head: bool = False, value_mix: dict | None = None,
+                 values_are_keys: bool = False, sink_logit: float | None = None):
         if n_q_heads % n_kv_heads:
             raise ValueError(f"{n_q_heads} query heads are not a multiple of {n_kv_heads} kv heads")
         if qk_norm not in (True, False, "unit_after", "whole"):
@@ -62,7 +66,14 @@ class GQAttention(Mixer):
         self.n_gate = 0 if gate is None else (self.n_q if self.gate_per_head else self.n_q * self.vd)
         self.plain_heads = (self.bias_names is None and not self.unit_after and not self.whole_norm and self.vd == self.hd
                             and self.chunk == 0 and self.scale == 0.0 and self.softcap == 0.0
-                            and sink is None and gate is None and value_mix is None)
+                            and sink is None and gate is None and value_mix is None and not values_are_keys
+                            and sink_logit is None)
+        self.values_are_keys = bool(values_are_keys)
+        if self.values_are_keys and (kv_shared or value_mix is not None or self.vd != self.hd):
+            raise ValueError("values that are the keys need keys of this mixer's own, of the values' size, and no mixing")
+        if sink is not None and sink_logit is not None:
+            raise ValueError("a softmax takes a learned sink or a fixed one, not both")
+        self.sink_logit = None if sink_logit is None else float(sink_logit)
         if value_mix is not None and kv_shared:
             raise ValueError("a mixer without values of its own cannot mix them")
         self.mix_key = None if value_mix is None else str(value_mix["key"])
@@ -77,8 +88,9 @@ class GQAttention(Mixer):
         n = self.names
         out = [ParamSpec(n["q"], (self.n_q * self.hd, self.width))]
         if not self.kv_shared:
-            out += [ParamSpec(n["k"], (self.n_kv * self.hd, self.width)),
-                    ParamSpec(n["v"], (self.n_kv * self.vd, self.width))]
+            out.append(ParamSpec(n["k"], (self.n_kv * self.hd, self.width)))
+            if not self.values_are_keys:
+                out.append(ParamSpec(n["v"], (self.n_kv * self.vd, self.width)))
         out.append(ParamSpec(n["o"], (self.width, self.n_q * self.vd)))
         if self.qk_norm:
             out.append(ParamSpec(n["q_norm"], (self.n_q * self.hd if self.whole_norm else self.hd,), init="norm"))
@@ -88,7 +100,9 @@ class GQAttention(Mixer):
             b = self.bias_names
             out.append(ParamSpec(b["q"], (self.n_q * self.hd,)))
             if not self.kv_shared:
-                out += [ParamSpec(b["k"], (self.n_kv * self.hd,)), ParamSpec(b["v"], (self.n_kv * self.vd,))]
+                out.append(ParamSpec(b["k"], (self.n_kv * self.hd,)))
+                if not self.values_are_keys:
+                    out.append(ParamSpec(b["v"], (self.n_kv * self.vd,)))
             if b.get("o"):
                 out.append(ParamSpec(b["o"], (self.width,)))
         if self.mix_name is not None:
@@ -99,6 +113,11 @@ class GQAttention(Mixer):
             out.append(ParamSpec(self.gate_name, (self.n_gate, self.width)))
         return out
 
+    @property
+    def _own_kv(self):
+        """The projections beside q that this mixer has."""
+        return () if self.kv_shared else ("k",) if self.values_are_keys else ("k", "v")
+
     def bind(self, tensors, rt):
         n = self.names
         if self.kv_shared and self.gate_name is None:
@@ -106,7 +125,7 @@ class GQAttention(Mixer):
         else:
             mats = [tensors.pop(n["q"])] if not self.kv_shared else [tensors[n["q"]]]
             if not self.kv_shared:
-                mats += [tensors.pop(n["k"]), tensors.pop(n["v"])]
+                mats += [tensors.pop(n[s]) for s in self._own_kv]
             if self.gate_name is not None:
                 mats.append(tensors.pop(self.gate_name))
             if len({t.dtype for t in mats}) > 1:
@@ -116,6 +135,8 @@ class GQAttention(Mixer):
             self.mix_lambda = float(tensors[self.mix_name].to(torch.float32).item())
         if self.sink_name is not None:
             self.sink = tensors[self.sink_name].to(torch.float32).contiguous()
+        elif self.sink_logit is not None:
+            self.sink = torch.full((self.n_q,), self.sink_logit, dtype=torch.float32, device=rt.device)
         self.w_o = tensors[n["o"]]
         if self.qk_norm:
             self.q_norm = tensors[n["q_norm"]]
@@ -124,7 +145,7 @@ class GQAttention(Mixer):
                 self.q_norm, self.k_norm = self.q_norm.float(), self.k_norm.float()
         if self.bias_names is not None:
             b = self.bias_names
-            parts = [tensors[b["q"]]] if self.kv_shared else [tensors.pop(b["q"]), tensors.pop(b["k"]), tensors.pop(b["v"])]
+            parts = [tensors[b["q"]]] if self.kv_shared else [tensors.pop(b[s]) for s in ("q", *self._own_kv)]
             if len({t.dtype for t in parts}) > 1:
                 parts = [t.float() for t in parts]
             self.b_qkv = torch.cat(parts, dim=0).contiguous()
@@ -187,7 +208,8 @@ class GQAttention(Mixer):
                               self.q_norm if self.qk_norm else None, self.k_norm if self.qk_norm else None, self.eps,
                               cos, sin, rot_dim, step.tok_pos, step.tok_seq, block_table, k_line, v_line,
                               write_kv=writes, q_out=q_out, bias=self.b_qkv, unit_norm_after=self.unit_after,
-                              v_head_dim=self.vd, whole_norm=self.whole_norm, pairs=pairs, **mix)
+                              v_head_dim=self.vd, whole_norm=self.whole_norm, pairs=pairs,
+                              values_are_keys=self.values_are_keys, **mix)
             rt.attention(step, q, o, self.n_q, self.n_kv, self.hd, k_line, v_line, block_table, self.window,
                          chunk=self.chunk, scale=self.scale, softcap=self.softcap, v_head_dim=self.vd, sink=self.sink)
             if self.gate_name is not None:

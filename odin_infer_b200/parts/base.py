@@ -141,6 +141,16 @@ class Normed:
         self.update, self.weight, self.eps, self.bias, self.center = update, weight, float(eps), bias, bool(center)
 
 
+class Streamed:
+    """An update of a residual that consists of several streams X[0] .. X[s-1] (`x` is [s, n, width]): with u the sum of
+    `update` (a tensor, `Biased`, `Several`, `Combined`), every stream becomes X[j] <- sum_i mix[i, j] X[i] + out[j] u, all of
+    them at once from the old ones.  mix: float32 [s, s] (from, to), out: float32 [s].  Only a norm that says `takes_streams`
+    may follow."""
+
+    def __init__(self, update, mix: torch.Tensor, out: torch.Tensor):
+        self.update, self.mix, self.out = update, mix, out
+
+
 def update_factor(pending) -> float:
     """The factor on a pending update (1 unless it is `Scaled`)."""
     return pending.factor if isinstance(pending, Scaled) else 1.0
@@ -150,7 +160,7 @@ def split_update(pending):
     """(delta, bias) of what a mixer or feed-forward answered: each a tensor or None (delta a list of
     tensors for `Several`).  The factor of a `Scaled` update is asked for with `update_factor`."""
     bias = None
-    if isinstance(pending, (Normed, Combined)):
+    if isinstance(pending, (Normed, Combined, Streamed)):
         return pending, None
     if isinstance(pending, Scaled):
         pending = pending.update
@@ -177,6 +187,7 @@ class Norm(Part):
     takes_several = False   # `delta` may be a list of up to three updates
     takes_scale = False     # takes a keyword `scale=`: x += scale * (the updates)
     takes_terms = False     # `delta` may be `Combined` or `Normed`
+    takes_streams = False   # x is [streams, n, width] and `delta` None or `Streamed`
 
     can_norm_updates = False  # may stand on a sublayer's output (has `as_update_norm`)
 
@@ -226,6 +237,13 @@ class FeedForward(Part):
         raise NotImplementedError
 
 
+class Connection(Part):
+    """How a sublayer's output joins a residual that is more than one stream."""
+
+    def join(self, update) -> Streamed:
+        raise NotImplementedError
+
+
 class Block(Part):
     def forward(self, rt, step, x: torch.Tensor, pending, entry: int):
         """x: residual stream (in place); pending: an update not yet added to it (None, [n, width]
@@ -261,7 +279,7 @@ class Head(Part):
 # ---------------------------------------------------------------- registries
 _REGISTRIES: dict[str, dict[str, Callable[..., Any]]] = {
     "mixer": {}, "feed_forward": {}, "norm": {}, "position_encoding": {}, "block": {}, "block_extra": {},
-    "embedding": {}, "head": {},
+    "connection": {}, "embedding": {}, "head": {},
 }
 
 

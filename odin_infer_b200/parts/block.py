@@ -1,8 +1,8 @@
 """How a layer's parts are arranged."""
 from __future__ import annotations
 
-from .base import (Block, Combined, Normed, PartSpec, ResidualAdded, Scaled, Several, build_part, register_part, split_update,
-                   update_factor)
+from .base import (Block, Combined, Normed, PartSpec, ResidualAdded, Scaled, Several, Streamed, build_part, register_part,
+                   split_update, update_factor)
 
 
 @register_part("block", "prenorm")
@@ -17,13 +17,25 @@ class PreNormBlock(Block):
     post_norm_mixer / post_norm_feed_forward: a norm on the sublayer's output before it is added (a plain RMSNorm or a
     layer norm), x -> x + Norm_b(Mixer(Norm(x))); with the norm "none" before the sublayer, x -> x + Norm_b(Mixer(x)).  The
     update travels as `Normed` to the norm that runs next, whose kernel sums the
-    sublayer's terms, norms them, adds and norms again.  No product then adds itself to x in its epilogue."""
+    sublayer's terms, norms them, adds and norms again.  No product then adds itself to x in its epilogue.
+
+    connect_mixer / connect_feed_forward: the residual is several streams (x is [streams, n, width]); each sublayer reads
+    what its norm forms of the streams, and its output joins them through that connection.  The update travels as `Streamed`
+    to the norm that runs next.  Both or neither; not together with norms on the outputs or extras."""
 
     def __init__(self, mixer: PartSpec, feed_forward: PartSpec | None, norm_mixer: PartSpec,
                  norm_feed_forward: PartSpec | None, extras: tuple = (), post_norm_mixer: PartSpec | None = None,
-                 post_norm_feed_forward: PartSpec | None = None):
+                 post_norm_feed_forward: PartSpec | None = None, connect_mixer: PartSpec | None = None,
+                 connect_feed_forward: PartSpec | None = None):
         if (feed_forward is None) != (norm_feed_forward is None):
             raise ValueError("a block has a feed-forward and its norm, or neither")
+        if connect_mixer is not None and (extras or post_norm_mixer is not None or post_norm_feed_forward is not None):
+            raise ValueError("a block whose residual is several streams takes no norms on its outputs and no extras")
+        if (connect_mixer is not None) != (connect_feed_forward is not None) and feed_forward is not None:
+            raise ValueError("a block's two sublayers join one residual: both through a connection, or neither")
+        self.connect_mixer = build_part("connection", connect_mixer) if connect_mixer is not None else None
+        self.connect_ffn = build_part("connection", connect_feed_forward) if (connect_mixer is not None
+                                                                              and feed_forward is not None) else None
         self.post_mixer = build_part("norm", post_norm_mixer) if post_norm_mixer is not None else None
         self.post_ffn = build_part("norm", post_norm_feed_forward) if (post_norm_feed_forward is not None
                                                                         and feed_forward is not None) else None
@@ -35,14 +47,19 @@ class PreNormBlock(Block):
         self.norm_mixer = build_part("norm", norm_mixer)
         self.norm_ffn = build_part("norm", norm_feed_forward) if norm_feed_forward is not None else None
         self.extras = [build_part("block_extra", e) for e in extras]
+        if self.connect_mixer is not None:
+            for norm in (self.norm_mixer, self.norm_ffn):
+                if norm is not None and not norm.takes_streams:
+                    raise TypeError(f"{type(norm).__name__} reads one residual stream, the block's residual is several")
 
     @property
     def mixer(self):
         return self._mixer
 
     def _parts(self):
-        return tuple(p for p in (self.norm_mixer, self._mixer, getattr(self, "post_mixer", None), self.norm_ffn, self.ffn,
-                                 getattr(self, "post_ffn", None), *self.extras) if p is not None)
+        return tuple(p for p in (self.norm_mixer, self._mixer, getattr(self, "post_mixer", None),
+                                 getattr(self, "connect_mixer", None), self.norm_ffn, self.ffn, getattr(self, "post_ffn", None),
+                                 getattr(self, "connect_ffn", None), *self.extras) if p is not None)
 
     def params(self):
         return [p for part in self._parts() for p in part.params()]
@@ -67,6 +84,8 @@ class PreNormBlock(Block):
         if isinstance(delta, (Normed, Combined)):
             if not norm.takes_terms:
                 raise TypeError(f"{type(norm).__name__} follows an update of several terms or with a norm of its own, and takes none")
+        if isinstance(delta, Streamed) and not norm.takes_streams:
+            raise TypeError(f"{type(norm).__name__} follows an update of several residual streams, and takes one")
         factor = update_factor(pending)
         if factor != 1.0:
             if not norm.takes_scale:
@@ -83,12 +102,16 @@ class PreNormBlock(Block):
         h = self._norm(self.norm_mixer, rt, x, pending)
         if self.post_mixer is not None:
             pending = self.post_mixer.as_update_norm(mixer.forward(rt, step, h, entry))
+        elif self.connect_mixer is not None:
+            pending = self.connect_mixer.join(mixer.forward(rt, step, h, entry))
         else:
             pending = mixer.forward(rt, step, h, entry, residual=x) if mixer.takes_residual else mixer.forward(rt, step, h, entry)
         if ffn is not None:
             h = self._norm(self.norm_ffn, rt, x, pending)
             if self.post_ffn is not None:
                 pending = self.post_ffn.as_update_norm(ffn.forward(rt, step, h))
+            elif self.connect_ffn is not None:
+                pending = self.connect_ffn.join(ffn.forward(rt, step, h))
             else:
                 pending = ffn.forward(rt, step, h, residual=x) if ffn.takes_residual else ffn.forward(rt, step, h)
         for extra in self.extras:

@@ -15,13 +15,18 @@ class TokenEmbedding(Embedding):
 
     pair = {"weight", "buckets", "mul_prev", "mul_cur"}: a second table of buckets + 1 rows is added, row
     (previous token * mul_prev + token * mul_cur) mod buckets, and its last row for a sequence's first token.  The previous
-    token is per-sequence state (`state_bytes`; the model tells the part which state entry is its own, `state_entry`)."""
+    token is per-sequence state (`state_bytes`; the model tells the part which state entry is its own, `state_entry`).
+
+    streams > 0: the residual is that many streams, [streams, n, width], all equal to the embedded rows."""
 
     graph_safe = True
 
     def __init__(self, vocab_size: int, width: int, weight: str, norm: PartSpec | None = None, scale: float = 1.0,
-                 pair: dict | None = None):
+                 pair: dict | None = None, streams: int = 0):
         self.vocab_size, self.width, self.weight_name, self.scale = vocab_size, width, weight, float(scale)
+        self.streams = int(streams)
+        if norm is not None and self.streams:
+            raise ValueError("an embedding with a norm of its own starts one residual stream")
         self.norm = build_part("norm", norm) if norm is not None else None
         self.table = None
         self.pair = None
@@ -56,7 +61,8 @@ class TokenEmbedding(Embedding):
         return {"elementwise"} | (self.norm.kernel_groups() if self.norm else set())
 
     def forward(self, rt, step):
-        x = rt.empty(step.n_rows, self.width, dtype=torch.float32)
+        shape = (self.streams, step.n_rows, self.width) if self.streams else (step.n_rows, self.width)
+        x = rt.empty(*shape, dtype=torch.float32)
         if self.pair is not None:
             before = step.state(self.state_entry).view(torch.int32)
             ops.embed_pair(self.table, self.pair_table, step.tok_ids, step.tok_seq, step.seq_start, step.seq_slots, before,

@@ -24,7 +24,7 @@ class LatentAttention(Mixer):
 
     sink: name of a tensor [n_heads], a learned logit per head whose exponential joins the softmax's denominator (no key, no
     value, not scaled).  gate: name of a matrix G [n_heads, width]; head h's output is multiplied by sigmoid(G h)_h as it
-    leaves W_uv.
+    leaves W_uv; with gate_per_head=False G is [n_heads * v_head_dim, width] and every element has a factor of its own.
 
     names: "dq", "dq_norm", "uq" (q_rank 0: "q" instead), "dkv", "dkv_norm", "uk", "uv", "o".  All products that read the
     input (W_dq or W_q, W_dkv, G) are fused into one.
@@ -35,7 +35,7 @@ class LatentAttention(Mixer):
 
     def __init__(self, width: int, n_heads: int, head_dim: int, rot_dim: int, v_head_dim: int, q_rank: int, kv_rank: int,
                  names: dict, position_encoding: str | None, eps: float, scale: float, window: int = 0,
-                 sink: str | None = None, gate: str | None = None):
+                 sink: str | None = None, gate: str | None = None, gate_per_head: bool = True):
         if min(width, n_heads, head_dim, v_head_dim, kv_rank) <= 0 or q_rank < 0 or rot_dim < 0 or rot_dim % 2:
             raise ValueError("latent attention needs positive sizes and an even rot_dim")
         if kv_rank + rot_dim > 512:
@@ -47,7 +47,7 @@ class LatentAttention(Mixer):
         self.q_rank, self.kv_rank, self.L = q_rank, kv_rank, kv_rank + rot_dim
         self.names, self.pe_name, self.eps = dict(names), position_encoding, float(eps)
         self.scale, self.window = float(scale), int(window)
-        self.sink_name, self.gate_name = sink, gate
+        self.sink_name, self.gate_name, self.gate_per_head = sink, gate, bool(gate_per_head)
         self.n_first = q_rank or n_heads * (head_dim + rot_dim)   # columns of the fused product before the kv latent's
         self.pe = None
         self.sink = self.q_norm = self.w_uq = self._dummy = None
@@ -65,7 +65,7 @@ class LatentAttention(Mixer):
         if self.sink_name is not None:
             out.append(ParamSpec(self.sink_name, (H,), init="logit"))
         if self.gate_name is not None:
-            out.append(ParamSpec(self.gate_name, (H, self.width)))
+            out.append(ParamSpec(self.gate_name, (H if self.gate_per_head else H * self.ev, self.width)))
         return out
 
     def bind(self, tensors, rt):

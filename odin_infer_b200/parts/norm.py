@@ -1,10 +1,11 @@
-"""Norms, fused with the residual add that precedes them: RMSNorm, layer norm, and none (the add alone)."""
+"""Norms, fused with the residual add that precedes them: RMSNorm (of one residual stream or of several), layer norm, and
+none (the add alone)."""
 from __future__ import annotations
 
 import torch
 
 from ..csrc import ops
-from .base import Combined, Norm, Normed, ParamSpec, Several, register_part
+from .base import Biased, Combined, Norm, Normed, ParamSpec, Several, Streamed, register_part
 
 
 def terms_of(update) -> list:
@@ -13,6 +14,8 @@ def terms_of(update) -> list:
         return list(update)
     if isinstance(update, Several):
         return [ops.Term(u) for u in update if u is not None]
+    if isinstance(update, Biased) and torch.is_tensor(update.update):
+        return [ops.Term(update.update, bias=update.bias)]
     if torch.is_tensor(update):
         return [ops.Term(update)]
     raise TypeError(f"an update of type {type(update).__name__} cannot be summed term by term")
@@ -103,6 +106,51 @@ class RMSNorm(Norm):
     def in_place(self, rt, x) -> None:
         """x (32-bit) <- its own norm."""
         ops.row_update(x, None, None, self.weight, self.eps, self.groups, x)
+
+
+@register_part("norm", "streams_rmsnorm")
+class StreamsRMSNorm(Norm):
+    """Reads a residual of several streams: o = w * u / sqrt(mean(u^2) + eps) of u = sum_i read[i] X[i], in 32-bit.
+
+    x is [streams, n, width]; a pending `Streamed` update is applied to the streams first, and the sum, the norm and that
+    update are one kernel.  read: name of a vector [streams] (None: the plain sum of the streams).  one_plus: as RMSNorm."""
+
+    graph_safe = True
+    takes_streams = True
+
+    def __init__(self, width: int, eps: float, weight: str, streams: int, read: str | None = None, one_plus: bool = False):
+        if not 1 <= streams <= ops.MAX_STREAMS:
+            raise ValueError(f"a residual has 1 to {ops.MAX_STREAMS} streams, got {streams}")
+        self.width, self.eps, self.weight_name, self.streams = width, float(eps), weight, int(streams)
+        self.read_name, self.one_plus = read, bool(one_plus)
+        self.weight = self.read = None
+
+    def params(self):
+        out = [ParamSpec(self.weight_name, (self.width,), init="near_zero" if self.one_plus else "norm")]
+        if self.read_name is not None:
+            out.append(ParamSpec(self.read_name, (self.streams,), init="unit"))
+        return out
+
+    def bind(self, tensors, rt):
+        self.weight = tensors[self.weight_name]
+        if self.one_plus:
+            self.weight = (self.weight.to(torch.float32) + 1.0).contiguous()
+        if self.read_name is not None:
+            self.read = tensors[self.read_name].to(torch.float32).contiguous()
+        else:
+            self.read = torch.ones(self.streams, dtype=torch.float32, device=rt.device)
+
+    def kernel_groups(self):
+        return {"streams"}
+
+    def forward(self, rt, x, delta, rows=None):
+        if delta is not None and not isinstance(delta, Streamed):
+            raise TypeError(f"a residual of several streams takes updates through a connection, not {type(delta).__name__}")
+        n = x.shape[1] if rows is None else rows.numel()
+        out = rt.empty(n, self.width)
+        terms, mix, add = ([], None, None) if delta is None else (terms_of(delta.update), delta.mix, delta.out)
+        ops.mix_streams(x, terms, mix, add, self.read, self.weight, self.eps, out, rows)
+        return out
 
 
 @register_part("norm", "layernorm")

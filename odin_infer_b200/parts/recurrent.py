@@ -175,6 +175,62 @@ class Retention(Mixer):
         return rt.linear(y, self.w_o, out_dtype=torch.float32, may_split=True)
 
 
+@register_part("mixer", "lightning")
+class Lightning(Mixer):
+    """Linear attention with one fixed decay per head between SiLUs, and one norm over all heads.
+
+    q = silu(W_q h), k = silu(W_k h) (heads x head_dim), v = silu(W_v h) (heads x v_head_dim), no biases, no positions and no
+    factor.  Per head, with the state S (head_dim x v_head_dim) zero at a sequence's start:
+
+        S_t = decay_h S_(t-1) + k_t v_t^T          o_t = S_t^T q_t
+
+    The heads side by side are divided by the root mean square of the whole row, multiplied by the weight `norm` and by
+    sigmoid(W_g h), and go through W_o.  The four projections of h are fused into one at load and leave it as 32-bit; SiLU,
+    decay and state are 32-bit.  names: "q", "k", "v", "g", "norm", "o"."""
+
+    graph_safe = True
+
+    def __init__(self, width: int, n_heads: int, head_dim: int, v_head_dim: int, decay, names: dict, eps: float = 1e-5):
+        decay = [float(d) for d in decay]
+        if len(decay) != n_heads:
+            raise ValueError(f"{n_heads} heads need as many decays, got {len(decay)}")
+        self.width, self.H, self.D, self.V, self.eps = width, n_heads, head_dim, v_head_dim, float(eps)
+        self.decay_values, self.names = decay, dict(names)
+
+    def params(self):
+        n, qk, vv = self.names, self.H * self.D, self.H * self.V
+        return [ParamSpec(n["q"], (qk, self.width)), ParamSpec(n["k"], (qk, self.width)),
+                ParamSpec(n["v"], (vv, self.width)), ParamSpec(n["g"], (vv, self.width)),
+                ParamSpec(n["norm"], (vv,), init="norm"), ParamSpec(n["o"], (self.width, vv))]
+
+    def bind(self, tensors, rt):
+        n = self.names
+        mats = [tensors.pop(n[s]) for s in ("q", "k", "v", "g")]
+        if len({t.dtype for t in mats}) > 1:
+            mats = [t.float() for t in mats]
+        self.w_qkvg = torch.cat(mats, dim=0).contiguous()
+        self.norm_w, self.w_o = tensors[n["norm"]], tensors[n["o"]]
+        # the heads' decays, rounded to 32-bit once
+        self.decay = torch.tensor(self.decay_values, dtype=torch.float64).to(torch.float32).contiguous().to(rt.device)
+
+    def state_bytes(self) -> int:
+        return 4 * self.H * self.D * self.V
+
+    def kernel_groups(self):
+        return {"recurrent", "state_space", "gemm_plain"}
+
+    def forward(self, rt, step, h, entry):
+        T, qk, vv = h.shape[0], self.H * self.D, self.H * self.V
+        qkvg = rt.linear(h, self.w_qkvg, out_dtype=torch.float32)
+        o = rt.empty(T, vv, dtype=torch.float32)
+        ops.linear_recurrence("fixed_silu", qkvg[:, :qk], qkvg[:, qk:2 * qk], None, qkvg[:, 2 * qk:2 * qk + vv], self.decay,
+                              self.decay, o, _f32_view(step.state(entry)), step.seq_start, step.seq_slots, step.n_seq_cap,
+                              self.H, self.D, self.V, block_len=_block_len(step), max_new=step.max_new)
+        y = rt.empty(T, vv)
+        ops.skip_gate_norm(o, None, None, self.V, qkvg[:, 2 * qk + vv:], self.norm_w, 1, self.eps, y, sigmoid_after=True)
+        return rt.linear(y, self.w_o, out_dtype=torch.float32, may_split=True)
+
+
 @register_part("mixer", "gated_linear_recurrence")
 class GatedLinearRecurrence(Mixer):
     """Linear attention whose forget gate also decides what is written (the HGRN2 form).

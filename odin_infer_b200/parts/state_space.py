@@ -1,7 +1,7 @@
 """State-space mixers, and a mixer of two branches that read the same input.
 
 `selective_scan` keeps a state row per channel (inner x state), `state_space_dual` a matrix per head (state x head_dim)
-with one decay per head and token; both keep the last taps - 1 inputs of their short causal convolution.  All of it
+with one decay per head and token, `gated_linear_unit` one number per channel; all keep the last taps - 1 inputs of their short causal convolution.  All of it
 lives in 32-bit floats in the engine's per-sequence state area (zeroed when a slot is handed out) and is carried from
 step to step; step sizes, decays, exponentials and the states are 32-bit whatever the element type of activations.
 """
@@ -10,7 +10,7 @@ from __future__ import annotations
 import torch
 
 from ..csrc import ops
-from .base import Combined, Mixer, ParamSpec, PartSpec, build_part, register_part
+from .base import Biased, Combined, Mixer, ParamSpec, PartSpec, build_part, register_part
 from .recurrent import _block_len, _f32_view
 
 
@@ -141,6 +141,82 @@ class StateSpaceDual(Mixer):
         return rt.linear(y, self.w_o, out_dtype=torch.float32, may_split=True)
 
 
+@register_part("mixer", "gated_linear_unit")
+class GatedLinearUnit(Mixer):
+    """A real-gated linear recurrent unit (one state number per channel) behind a short convolution, times a second branch.
+
+    y = gelu_tanh(W_y h + b_y) and u = conv(W_x h + b_x), both `inner` wide; conv is causal, per channel (`taps` taps, the last
+    one the current token's, a bias, zeros before the start, no activation).  u is cut into `blocks` equal parts; part b gives
+    r = sigmoid(Ra[b] u_b + ra_b[b]) and i = sigmoid(Ri[b] u_b + ri_b[b]).  Per channel, with softplus(lam) and all that
+    follows in 32-bit:
+
+        log a = -sharpness r softplus(lam);     S <- a S + sqrt(1 - a^2) i u
+
+    from S = 0 at a sequence's start, and S * y goes through W_o.  The state keeps S and the convolution's last taps - 1
+    inputs (biases included).  W_y and W_x are one product; a block's two gate matrices are one product per block.
+    names: "y", "y_bias", "x", "x_bias", "conv", "conv_bias", "ra", "ra_bias", "ri", "ri_bias" ([blocks, m, m] as
+    [out, in], and [blocks, m]), "lam", "o"."""
+
+    graph_safe = True
+
+    def __init__(self, width: int, inner: int, blocks: int, taps: int, names: dict, sharpness: float = 8.0):
+        if min(width, inner, blocks, taps) < 1 or inner % blocks:
+            raise ValueError(f"a gated linear unit needs positive sizes and channels ({inner}) a multiple of blocks ({blocks})")
+        self.width, self.inner, self.blocks, self.taps = width, inner, blocks, taps
+        self.m, self.sharpness, self.names = inner // blocks, float(sharpness), dict(names)
+
+    def params(self):
+        n, m = self.names, self.m
+        out = []
+        for s in "yx":
+            out += [ParamSpec(n[s], (self.inner, self.width)), ParamSpec(n[s + "_bias"], (self.inner,), init="near_zero")]
+        out += [ParamSpec(n["conv"], (self.inner, self.taps), init="unit"), ParamSpec(n["conv_bias"], (self.inner,), init="near_zero")]
+        for s in ("ra", "ri"):
+            out += [ParamSpec(n[s], (self.blocks, m, m)), ParamSpec(n[s + "_bias"], (self.blocks, m), init="near_zero")]
+        return out + [ParamSpec(n["lam"], (self.inner,), init="decay"), ParamSpec(n["o"], (self.width, self.inner))]
+
+    def bind(self, tensors, rt):
+        n, m = self.names, self.m
+
+        def pair(a, b, dim):
+            a, b = tensors.pop(n[a]), tensors.pop(n[b])
+            return torch.cat([a, b] if a.dtype == b.dtype else [a.float(), b.float()], dim=dim).contiguous()
+        self.w_yx, self.w_o = pair("y", "x", 0), tensors[n["o"]]
+        self.y_bias, self.x_bias = _as_f32(tensors[n["y_bias"]], tensors[n["x_bias"]])
+        self.conv_w, self.conv_b = tensors[n["conv"]].contiguous(), tensors[n["conv_bias"]].contiguous()
+        # per block [r rows | i rows], in both orders (see Runtime.heads_linear); the biases as the products' columns lie
+        gates = pair("ra", "ri", 1)
+        self.w_gates = (gates.transpose(1, 2).contiguous(), gates)
+        self.gate_bias = torch.cat([t.view(self.blocks, m) for t in _as_f32(tensors[n["ra_bias"]], tensors[n["ri_bias"]])], dim=1).contiguous()
+        lam = tensors[n["lam"]].to(torch.float64)
+        self.log_decay = (-self.sharpness * torch.nn.functional.softplus(lam, threshold=40.0)).to(torch.float32).contiguous()
+
+    def state_bytes(self) -> int:
+        return 4 * (self.inner + (self.taps - 1) * self.inner)
+
+    def kernel_groups(self):
+        return {"state_space", "gated_unit", "latent", "moe_tc", "gemm_plain"}
+
+    def forward(self, rt, step, h, entry):
+        T, n = h.shape[0], self.inner
+        state = _f32_view(step.state(entry))
+        S, window = state[:, :n], state[:, n:]
+        yx = rt.linear(h, self.w_yx)
+        u = rt.empty(T, n)
+        ops.causal_conv(yx[:, n:], self.conv_w, self.conv_b, False, window, step.tok_seq, step.seq_start, step.seq_slots,
+                        step.n_seq_cap, u, single_rows=step.all_single, in_bias=self.x_bias)
+        out = rt.empty(T, n)
+        if step.all_single:
+            ops.gated_unit_step(u, self.w_gates[0], self.gate_bias, self.log_decay, yx[:, :n], self.y_bias, S, out,
+                                step.tok_seq, step.seq_slots)
+        else:
+            raw = rt.empty(T, 2 * n, dtype=torch.float32)
+            rt.heads_linear(u, self.m, self.w_gates, raw, 2 * self.m)
+            ops.gated_unit_scan(u, raw, self.gate_bias, self.log_decay, yx[:, :n], self.y_bias, S, out, step.seq_start,
+                                step.seq_slots, step.n_seq_cap, step.max_new)
+        return rt.linear(out, self.w_o, out_dtype=torch.float32, may_split=True)
+
+
 @register_part("mixer", "side_by_side")
 class SideBySide(Mixer):
     """Two mixers that read the same input; the update is left_scale * f_l(left) + right_scale * f_r(right), f the
@@ -214,8 +290,10 @@ class SideBySide(Mixer):
     def forward(self, rt, step, h, entry):
         out = Combined()
         for m, scale, w in zip(self._both(), self.scales, self.norm_w):
-            u = m.forward(rt, step, h, entry)
+            u, bias = m.forward(rt, step, h, entry), None
+            if isinstance(u, Biased):
+                u, bias = u.update, u.bias
             if not torch.is_tensor(u):
                 raise TypeError(f"{type(m).__name__} beside another mixer must answer a plain update, got {type(u).__name__}")
-            out.append(ops.Term(u, scale, None, w, self.eps))
+            out.append(ops.Term(u, scale, None, w, self.eps, bias))
         return out
