@@ -1371,6 +1371,251 @@ def fugavik_workload(steps: int, warmup: int) -> int:
     return 0
 
 
+# --------------------------------------------------------------------------------------------------------------
+# --workload bafilorn: the Bafilorn design beside the Fugavik design (the closest: latent attention, a matrix-state recurrence,
+# grouped attention, dense feed-forwards with relu squared)
+# --------------------------------------------------------------------------------------------------------------
+BAFILORN_SIZES = {
+    # the Fugavik sizes' width, layers, vocabulary, attention heads and dense feed-forwards (here in every layer of both
+    # designs), latent rows of 64 + 64, recurrences over as many heads of 128 x 128; gated units of the model's width in
+    # blocks of 256 channels; four residual streams
+    "2048": dict(FUGAVIK_SIZES["2048"], streams=4, unit=2048, unit_blocks=8, chunk=1024, lat_rank=64),
+    "4096": dict(FUGAVIK_SIZES["4096"], streams=4, unit=4096, unit_blocks=16, chunk=1024, lat_rank=64),
+}
+
+
+def bafilorn_config(z: dict) -> dict:
+    lat = {"heads": z["lat_heads"], "dim": z["lat_dim"], "rot_dim": z["rot_dim"], "vdim": z["lat_v"], "q_rank": z["q_rank"],
+           "kv_rank": z["lat_rank"], "scale": (z["lat_dim"] + z["rot_dim"]) ** -0.5, "rot": {"dims": z["rot_dim"], "base": 500000.0}}
+    H = z["delta_heads"]
+    lig = {"heads": H, "dim": z["delta_dim"], "vdim": z["delta_v"],
+           "decay": [math.exp(-1.0 / (8.0 * 2.0 ** (8.0 * i / max(H - 1, 1)))) for i in range(H)]}   # memories of 8 to 2,048 tokens
+    par = {"left": {"heads": z["heads"], "kv_heads": z["kv"], "dim": z["hd"], "vdim": z["hd"], "scale": z["hd"] ** -0.5,
+                    "mask": {"size": z["chunk"]},
+                    "rot": {"dims": z["hd"] // 2, "base": 500000.0,
+                            "scaling": {"factor": 8.0, "original": 4096, "fast": 24.0, "slow": 1.5}}},
+           "right": {"width": z["unit"], "blocks": z["unit_blocks"], "conv": 3}}
+    cycle = [("lightning", lig), ("parallel", par), ("latent_attention", lat), ("parallel", par)]
+    layers = [{"type": t, "mixer": m, "mlp": {"kind": "dense", "ff": z["dense"]}} for t, m in (cycle[i % 4] for i in range(z["layers"]))]
+    return {"architecture": "Bafilorn", "vocab": z["vocab"], "width": z["width"], "streams": z["streams"], "norm": {"eps": 1e-5},
+            "embedding": {"scale": 1.5, "bigram": {"buckets": 99991, "mul_prev": 131, "mul_cur": 31}}, "layers": layers}
+
+
+def bafilorn_kernels(z: dict, T: int, peaks: dict) -> dict:
+    """Every kernel that the design adds (or runs with options of its own), alone at this size for T token rows (one
+    prompt of T tokens, or T sequences of one token after 512), beside the like kernel of the closest existing path:
+    microseconds, and algorithmic bytes (or FLOPs) over the time as a fraction of the measured peaks."""
+    import torch
+    from odin_infer_b200.csrc import ops
+    from odin_infer_b200.engine import runtime as R
+    dev, bf = "cuda:0", torch.bfloat16
+    flush = torch.empty(256 << 20, dtype=torch.uint8, device=dev)
+    d = z["width"]
+    decode = T <= 64
+    out = {}
+
+    def replayed(fn, flush, reps=5, inner=20):
+        fn()
+        torch.cuda.synchronize()
+        graph = torch.cuda.CUDAGraph()
+        with torch.cuda.graph(graph):
+            for _ in range(inner):
+                fn()
+        return _timed(graph.replay, flush, reps) / inner
+    timed = replayed if decode else _timed
+
+    def note(name, us, nbytes=None, flops=None, **more):
+        rec = {"us": round(us, 2)}
+        if nbytes is not None:
+            rec["of_hbm"] = round(nbytes / (us * 1e-6) / 1e9 / peaks["hbm_gbs"], 3)
+        if flops is not None:
+            rec["tflops"] = round(flops / (us * 1e-6) / 1e12, 2)
+        rec.update(more)
+        out[name] = rec
+    rt = R.Runtime(dev, bf)
+    torch.manual_seed(0)
+    ctx = 512 if decode else 0
+    n_seq = T if decode else 1
+    per_seq = (ctx + 1 + 63) // 64 if decode else (T + 63) // 64
+    n_pages = n_seq * per_seq
+    bt = torch.arange(n_pages, dtype=torch.int32, device=dev).reshape(n_seq, per_seq).contiguous()
+    pos = torch.full((T,), ctx, dtype=torch.int32, device=dev) if decode else torch.arange(T, dtype=torch.int32, device=dev)
+    seq = torch.arange(T, dtype=torch.int32, device=dev) if decode else torch.zeros(T, dtype=torch.int32, device=dev)
+    starts = torch.arange(0, T + 1, 1 if decode else T, dtype=torch.int32, device=dev)
+    slots = torch.arange(n_seq, dtype=torch.int32, device=dev)
+    w1, w2 = torch.randn(d, device=dev), torch.randn(d, device=dev)
+    hb = torch.empty(T, d, dtype=bf, device=dev)
+    d1, d2 = torch.randn(T, d, device=dev), torch.randn(T, d, device=dev)
+    # the residual: one stream and its norm, beside several streams, their mix, the read sum and its norm
+    x = torch.randn(T, d, device=dev)
+    note("add + RMSNorm of an update (fugavik's neighbour meropel)", timed(lambda: ops.combine_add(x, [ops.Term(d1)], None, 0.0, w1, 1e-5, hb), flush), nbytes=T * d * 14)
+    note("two terms each with a norm of its own, the add, the next norm (meropel)", timed(
+        lambda: ops.combine_add(x, [ops.Term(d1, 0.5, None, w1, 1e-5), ops.Term(d2, 0.5, None, w2, 1e-5)], None, 0.0, w1, 1e-5, hb), flush), nbytes=T * d * 18)
+    for s in (2, 4):
+        xs = torch.randn(s, T, d, device=dev)
+        mix, add, read = torch.full((s, s), 1.0 / s, device=dev), torch.randn(s, device=dev), torch.randn(s, device=dev)
+        note(f"{s} streams: an update joins, the next norm", timed(
+            lambda: ops.mix_streams(xs, [ops.Term(d1)], mix, add, read, w1, 1e-5, hb), flush), nbytes=T * d * (8 * s + 6))
+        note(f"{s} streams: two terms each with a norm of its own join, the next norm", timed(
+            lambda: ops.mix_streams(xs, [ops.Term(d1, 0.5, None, w1, 1e-5, w2), ops.Term(d2, 0.5, None, w2, 1e-5)], mix, add, read, w1, 1e-5, hb), flush),
+            nbytes=T * d * (8 * s + 10))
+    # the embedding with the pair's row, into one stream and into several
+    V, buckets = z["vocab"], 99991
+    table, pairs = torch.randn(V, d, device=dev).to(bf), torch.randn(buckets + 1, d, device=dev).to(bf)
+    tok = torch.randint(0, V, (T,), dtype=torch.int32, device=dev)
+    before = torch.zeros(n_seq, 64, dtype=torch.int32, device=dev)
+    note("embedding plus the row of the pair (meropel)", timed(
+        lambda: ops.embed_pair(table, pairs, tok, seq, starts, slots, before, n_seq, buckets, 131, 31, x, single_rows=decode), flush), nbytes=T * d * 8)
+    xs = torch.empty(z["streams"], T, d, device=dev)
+    note(f"embedding plus the row of the pair, into {z['streams']} streams", timed(
+        lambda: ops.embed_pair(table, pairs, tok, seq, starts, slots, before, n_seq, buckets, 131, 31, xs, 1.5, single_rows=decode), flush), nbytes=T * d * (4 + 4 * z["streams"]))
+    # head preparation with biases and a partial rotation; the values are the keys
+    Hq, Hkv, hd = z["heads"], z["kv"], z["hd"]
+    kc = (torch.randn(n_pages, Hkv, 64, hd, device=dev) * 0.3).to(bf)
+    vc = (torch.randn(n_pages, Hkv, 64, hd, device=dev) * 0.3).to(bf)
+    qkv = torch.randn(T, (Hq + 2 * Hkv) * hd, device=dev).to(bf)
+    bias = torch.randn((Hq + 2 * Hkv) * hd, device=dev).to(bf)
+    ch = torch.randn(max(T, ctx + 1), hd // 4, device=dev)
+    q_out = torch.empty(T, Hq * hd, dtype=bf, device=dev)
+    note("head preparation with biases and a unit norm after a partial rotation (tovalix)", timed(
+        lambda: ops.head_prep(qkv, Hq, Hkv, hd, None, None, 1e-5, ch, ch, hd // 2, pos, seq, bt, kc, vc, q_out=q_out, bias=bias, unit_norm_after=True), flush),
+        nbytes=T * (Hq + 2 * Hkv) * hd * 4)
+    qk, qk_bias = qkv[:, :(Hq + Hkv) * hd].contiguous(), bias[:(Hq + Hkv) * hd].contiguous()
+    note("head preparation with biases, a partial rotation, values that are the keys", timed(
+        lambda: ops.head_prep(qk, Hq, Hkv, hd, None, None, 1e-5, ch, ch, hd // 2, pos, seq, bt, kc, vc, q_out=q_out, bias=qk_bias, values_are_keys=True), flush),
+        nbytes=T * (2 * Hq + 3 * Hkv) * hd * 2)
+    # attention over chunks with one added to the denominator, and over latent rows
+    H, e, r, ev, L, qr = z["lat_heads"], z["lat_dim"], z["rot_dim"], z["lat_v"], z["lat_rank"] + z["rot_dim"], z["q_rank"]
+    rows = (torch.randn(n_pages, 1, 64, L, device=dev) * 0.3).to(bf)
+    qf, of = torch.randn(T, H * L, device=dev).to(bf), torch.empty(T, H * L, dtype=bf, device=dev)
+    zero = torch.zeros(Hq, device=dev)
+    C = z["chunk"]
+    pairs_in = sum(min(C, T - c) * (min(C, T - c) + 1) // 2 for c in range(0, T, C))
+    for name, qq, nq, nkv, dim, k_, v_, chunk, sk in (
+            (" (fugavik, no sink)", q_out, Hq, Hkv, hd, kc, vc, 0, None), (f", chunks of {C}, one added to the denominator", q_out, Hq, Hkv, hd, kc, vc, C, zero),
+            (" over latent rows", qf, H, 1, L, rows, rows, 0, None)):
+        oo = torch.empty_like(qq)
+        if decode:
+            n_split = R.decode_key_splits(T, nkv, ctx + 1)
+            scratch = torch.empty(ops.attention_decode_scratch(T, nq, dim, n_split), dtype=torch.float32, device=dev)
+            note("decode attention over 512 keys" + name, timed(
+                lambda: ops.attention_decode(qq, oo, nq, nkv, dim, k_, v_, pos, seq, bt, 0, scratch, n_split, chunk, dim ** -0.5, 0.0, sk), flush),
+                nbytes=T * (ctx + 1) * nkv * dim * 2 * (2 if k_ is not v_ else 1))
+        else:
+            lens = torch.tensor([T], dtype=torch.int32, device=dev)
+            note("prompt attention" + name, timed(
+                lambda: ops.attention_prefill(qq, oo, 1, T, nq, nkv, dim, k_, v_, starts, lens, bt, 0, chunk, dim ** -0.5, 0.0, sk), flush),
+                flops=4.0 * nq * dim * (pairs_in if chunk else T * (T + 1) / 2))
+    gate = torch.randn(T, Hq * hd, device=dev).to(bf)
+    og = torch.randn(T, Hq * hd, device=dev).to(bf)
+    note("a sigmoid gate per element on attention's output (nufupel)", timed(lambda: ops.sigmoid_gate(og, gate, Hq, hd, False), flush), nbytes=T * Hq * hd * 6)
+    # around latent attention: the latents' norms and the cached row, the products per head without and with a gate per element
+    down = torch.randn(T, qr + L + H * ev, device=dev).to(bf)
+    qn, cn = torch.ones(qr, dtype=bf, device=dev), torch.ones(z["lat_rank"], dtype=bf, device=dev)
+    cr, cq = torch.randn(max(T, ctx + 1), r // 2, device=dev), torch.empty(T, qr, dtype=bf, device=dev)
+    note("latent preparation (both norms, rotation, cache row; nikonex)", timed(
+        lambda: ops.latent_prep(down[:, :qr + L], qr, z["lat_rank"], r, True, qn, cn, 1e-5, cq, cr, cr, pos, seq, bt, rows), flush), nbytes=T * (qr + L) * 4)
+    w_uv = (torch.randn(H, L, ev, device=dev) / L ** 0.5).to(bf)
+    ov, uv = torch.empty(T, H * ev, dtype=bf, device=dev), (w_uv, w_uv.transpose(1, 2).contiguous())
+    vb = T * H * (L + ev) * 2 + w_uv.numel() * 2
+    note("values from the latent, times the head's gate (fugavik)", timed(lambda: rt.heads_linear(of, L, uv, ov, ev, gate=down[:, qr:qr + H]), flush),
+         flops=2.0 * T * H * L * ev, nbytes=vb)
+    note("values from the latent, times a gate per element", timed(lambda: rt.heads_linear(of, L, uv, ov, ev, gate=down[:, qr + L:]), flush),
+         flops=2.0 * T * H * L * ev, nbytes=vb + T * H * ev * 2)
+    # the recurrence between SiLUs beside retention's, and the norm over all heads beside the norm per head
+    RH, dk, dv = z["delta_heads"], z["delta_dim"], z["delta_v"]
+    blocks = dict(block_len=128, max_new=T) if not decode else {}
+    tag = " in blocks of 128 tokens" if not decode else ""
+    state = torch.zeros(n_seq, RH * dk * dv, device=dev)
+    qkvg = torch.randn(T, RH * (2 * dk + 2 * dv), device=dev)
+    q, k, v, g = qkvg[:, :RH * dk], qkvg[:, RH * dk:2 * RH * dk], qkvg[:, 2 * RH * dk:RH * (2 * dk + dv)], qkvg[:, RH * (2 * dk + dv):]
+    ro, decay = torch.empty(T, RH * dv, device=dev), torch.full((RH,), 0.99, device=dev)
+    for mode, name in (("fixed", "recurrence with a fixed decay (nikonex)"), ("fixed_silu", "recurrence with a fixed decay between SiLUs")):
+        state.zero_()
+        note(f"{name}, {RH} heads of {dk} x {dv}" + tag, timed(
+            lambda: ops.linear_recurrence(mode, q, k, None, v, decay, decay, ro, state, starts, slots, n_seq, RH, dk, dv, **blocks), flush),
+            nbytes=4 * (T * 2 * RH * (dk + dv) + 2 * n_seq * RH * dk * dv), flops=T * RH * 4.0 * dk * dv)
+    y, wn, wh = torch.empty(T, RH * dv, dtype=bf, device=dev), torch.ones(RH * dv, dtype=bf, device=dev), torch.ones(dv, dtype=bf, device=dev)
+    note("heads' norm with a shared weight times silu(gate) (fugavik)", timed(lambda: ops.head_unit_scale(ro, wh, False, g, 1e-5, y, RH, dv), flush), nbytes=T * RH * dv * 10)
+    note("silu(gate) and a norm in groups (meropel)", timed(lambda: ops.skip_gate_norm(ro, None, None, dv, g, wn, 8, 1e-5, y), flush), nbytes=T * RH * dv * 10)
+    note("one norm over all heads times sigmoid(gate)", timed(
+        lambda: ops.skip_gate_norm(ro, None, None, dv, g, wn, 1, 1e-5, y, sigmoid_after=True), flush), nbytes=T * RH * dv * 10)
+    # the gated unit: its convolution, the gates' products, the recurrence; beside the selective scan's
+    n, nb = z["unit"], z["unit_blocks"]
+    m = n // nb
+    yx = torch.randn(T, 2 * n, device=dev).to(bf)
+    cw, cb, xb = torch.randn(n, 3, device=dev).to(bf), torch.randn(n, device=dev).to(bf), torch.randn(n, device=dev)
+    cs, u = torch.zeros(n_seq, 2 * n, device=dev), torch.empty(T, n, dtype=bf, device=dev)
+    cbytes = T * n * 4 + 2 * n_seq * 2 * n * 4
+    note("causal convolution of 3 taps, SiLU, its memory (meropel)", timed(
+        lambda: ops.causal_conv(yx[:, n:], cw, cb, True, cs, seq, starts, slots, n_seq, u, single_rows=decode), flush), nbytes=cbytes)
+    note("causal convolution of 3 taps with a bias on its inputs, its memory", timed(
+        lambda: ops.causal_conv(yx[:, n:], cw, cb, False, cs, seq, starts, slots, n_seq, u, single_rows=decode, in_bias=xb), flush), nbytes=cbytes)
+    wg = (torch.randn(nb, 2 * m, m, device=dev) / m ** 0.5).to(bf)
+    wg = (wg.transpose(1, 2).contiguous(), wg)
+    gb, ld, yb = torch.randn(nb, 2 * m, device=dev), -torch.rand(n, device=dev), torch.randn(n, device=dev)
+    S, res = torch.zeros(n_seq, n, device=dev), torch.empty(T, n, dtype=bf, device=dev)
+    N = 16
+    xz, dt = torch.randn(T, 2 * n, device=dev).to(bf), torch.randn(T, n, device=dev)
+    bc, a_log = torch.randn(T, 2 * N, device=dev), torch.randn(n, N, device=dev) * 0.5
+    dd, dtb, st = torch.randn(n, device=dev), torch.randn(n, device=dev) - 2, torch.zeros(n_seq, n * N, device=dev)
+    note(f"selective scan of {n} channels of {N} states with skip and gate (meropel)" + tag, timed(
+        lambda: ops.selective_scan(u, dt, dtb, bc[:, :N], bc[:, N:], a_log, dd, xz[:, n:], st, res, starts, slots, n_seq, **blocks), flush),
+        nbytes=T * n * 10 + T * 2 * N * 4 + 2 * n_seq * n * N * 4 + n * N * 4)
+    if decode:
+        note(f"gated unit of {n} channels: gate products, recurrence, output", timed(
+            lambda: ops.gated_unit_step(u, wg[0], gb, ld, yx[:, :n], yb, S, res, seq, slots), flush), nbytes=wg[0].numel() * 2 + T * n * 14)
+    raw = torch.empty(T, 2 * n, device=dev)
+    note("gate products, a product per block", timed(lambda: rt.heads_linear(u, m, wg, raw, 2 * m), flush), flops=2.0 * T * 2 * n * m,
+         nbytes=T * n * 10 + wg[0].numel() * 2)
+    note(f"gated unit's recurrence over {n} channels, with its output", timed(
+        lambda: ops.gated_unit_scan(u, raw, gb, ld, yx[:, :n], yb, S, res, starts, slots, n_seq, 1 if decode else T), flush), nbytes=T * n * 14)
+    torch.cuda.synchronize()
+    return out
+
+
+def bafilorn_workload(steps: int, warmup: int) -> int:
+    """The Bafilorn design at two sizes that resemble a real model's layers, beside the Fugavik design of the same width,
+    layers, vocabulary and feed-forwards (random weights): a prompt of 2,048 tokens in one step, decoding at batch 8
+    after 512-token prompts (device-timed), and every kernel of the design alone beside its like."""
+    import torch
+    from odin_infer_b200 import Engine, Engine_Opts
+    from odin_infer_b200.config import config_from_dict
+    from odin_infer_b200.csrc import ops
+    peaks, peak_source = load_peaks()
+    result = {"metric": "Bafilorn beside Fugavik at equal sizes: prompt of 2,048 tokens, decode at batch 8 (512-token prompts), "
+                        "bf16, random weights", "peak_source": peak_source, "sizes": {}}
+    steps = min(steps, 64)
+    for name, z in BAFILORN_SIZES.items():
+        entry = {}
+        beside = fugavik_config(z)
+        for l in beside["layers"]:
+            l["mlp"] = {"kind": "dense", "ff": z["dense"]}
+        for model, raw in (("bafilorn", bafilorn_config(z)), ("fugavik", beside)):
+            need = PROMPT + warmup + steps + 72
+            engine = Engine.random(config_from_dict(raw), WEIGHT_SEED, Engine_Opts(
+                max_ctx=CONTEXT, max_tokens=max(8 * ((need + 63) // 64 * 64), PREFILL_TOKENS + 64), max_batch=8,
+                dtype="bfloat16", verbose=False))
+            ms_pf = run_prefill(engine, z["vocab"])
+            tps, ms_step, _, launches = run_decode(engine, 8, steps, warmup, z["vocab"])
+            entry[model] = {"layers": z["layers"], "weights_gib": round(engine.weight_bytes / 2 ** 30, 2),
+                            "prefill_2048": {"ms": round(ms_pf, 3), "tokens_per_s": round(PREFILL_TOKENS / ms_pf * 1e3)},
+                            "decode_b8": {"ms_per_step": round(ms_step, 4), "tokens_per_s": round(tps, 1),
+                                          "launches_per_step": launches // steps}}
+            engine.destroy()
+            del engine
+            torch.cuda.empty_cache()
+        entry["kernels_prompt_2048_rows"] = bafilorn_kernels(z, PREFILL_TOKENS, peaks)
+        entry["kernels_decode_8_rows"] = bafilorn_kernels(z, 8, peaks)
+        result["sizes"][name] = entry
+    ops.gemm_tc_check()
+    ops.attention_prefill_check()
+    ops.attention_decode_check()
+    ops.moe_tc_check()
+    print(json.dumps(result))
+    return 0
+
+
 def main() -> int:
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1382,14 +1627,14 @@ def main() -> int:
     ap.add_argument("--no-points", action="store_true", help="skip the batch 1 / 64 points and the prefill")
     ap.add_argument("--no-graphs", action="store_true", help="launch the decode step's kernels one by one (for profilers)")
     ap.add_argument("--no-e2e", action="store_true", help="skip the end-to-end run (for profilers)")
-    ap.add_argument("--workload", default="8b", choices=["8b", "1.7b-mixed", "32b-long", "tovalix", "nufupel", "nikonex", "meropel", "fugavik"],
+    ap.add_argument("--workload", default="8b", choices=["8b", "1.7b-mixed", "32b-long", "tovalix", "nufupel", "nikonex", "meropel", "fugavik", "bafilorn"],
                     help="8b: the contract's run (default).  The others are further workloads of the baseline's list and "
                          "print a line of their own: 1.7b-mixed = Qwen3-1.7B shape, 64 prompts of 16..2048 tokens, 128 new "
                          "tokens each; 32b-long = Qwen3-32B shape, a 2,048-token prompt, decoding 1 and 8 sequences at context 8192; "
                          "tovalix = the Tovalix design beside the Qwen3 decoder at equal sizes, and its kernels alone; "
                          "nufupel = the same for the Nufupel design; nikonex = the Nikonex design beside Nufupel at equal sizes, "
                          "and its kernels alone; meropel, fugavik = the Meropel or the Fugavik design beside Nikonex at equal sizes, and its "
-                         "kernels alone")
+                         "kernels alone; bafilorn = the Bafilorn design beside Fugavik with dense feed-forwards, and its kernels alone")
     args = ap.parse_args()
 
     if args.impl == "reference":
@@ -1411,6 +1656,8 @@ def main() -> int:
         return meropel_workload(args.steps, warmup)
     if args.workload == "fugavik":
         return fugavik_workload(args.steps, warmup)
+    if args.workload == "bafilorn":
+        return bafilorn_workload(args.steps, warmup)
     if args.workload != "8b":
         return other_workload(args.workload)
 

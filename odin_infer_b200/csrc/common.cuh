@@ -99,6 +99,9 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 //     still reads); before it a kernel may touch only what no kernel of the step writes:
 //     weights and constant tables, the step's integer tables (the host copies them to the
 //     device before the step's first kernel), and the cache as earlier steps left it;
+//   * a load through a const __restrict__ pointer counts as invariant, and the compiler may move it ahead of pdl_wait()
+//     (it does where the same condition guards a load of weights there): what an earlier kernel writes is read through
+//     pointers without __restrict__ wherever loads of weights stand before the wait;
 //   * every kernel launched this way calls pdl_wait(), so completion stays in stream
 //     order.  Set ODIN_PDL=0 in the environment to launch in plain stream order.
 // ---------------------------------------------------------------------------

@@ -24,14 +24,35 @@ struct HeadGate {
     __device__ __forceinline__ float element(int t, int h, int n, int N) const {
         return (p == nullptr || !per_element) ? 1.0f : sigmoid_at(t, h * N + n);
     }
-    __device__ __forceinline__ float4 sigmoid4_at(int t, int col) const {
-        float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
+    // one column of TOK tokens from t0 on (those before T)
+    template <int TOK>
+    __device__ __forceinline__ void columns(int t0, int T, int col, float (&f)[TOK]) const {
+#pragma unroll
+        for (int u = 0; u < TOK; ++u) f[u] = 0.f;
+        for (int s = 0; s < n_split; ++s) {
+#pragma unroll
+            for (int u = 0; u < TOK; ++u) {
+                const size_t at = (size_t)s * split_stride + (size_t)(t0 + u) * row_stride + col;
+                if (t0 + u < T) f[u] += is_bf16 ? __bfloat162float(((const bf16*)p)[at]) : ((const float*)p)[at];
+            }
+        }
+#pragma unroll
+        for (int u = 0; u < TOK; ++u) f[u] = 1.0f / (1.0f + expf(-f[u]));
+    }
+    // 32 columns from col on, loads together (aligned4)
+    __device__ __forceinline__ void sigmoid32(int t, int col, float (&f)[32]) const {
+#pragma unroll
+        for (int q = 0; q < 32; ++q) f[q] = 0.f;
         for (int s = 0; s < n_split; ++s) {
             const size_t at = (size_t)s * split_stride + (size_t)t * row_stride + col;
-            const float4 v = is_bf16 ? ld4((const bf16*)p + at) : ld4((const float*)p + at);
-            z.x += v.x; z.y += v.y; z.z += v.z; z.w += v.w;
+#pragma unroll
+            for (int q = 0; q < 32; q += 4) {
+                const float4 v = is_bf16 ? ld4((const bf16*)p + at + q) : ld4((const float*)p + at + q);
+                f[q] += v.x; f[q + 1] += v.y; f[q + 2] += v.z; f[q + 3] += v.w;
+            }
         }
-        return make_float4(1.0f / (1.0f + expf(-z.x)), 1.0f / (1.0f + expf(-z.y)), 1.0f / (1.0f + expf(-z.z)), 1.0f / (1.0f + expf(-z.w)));
+#pragma unroll
+        for (int q = 0; q < 32; ++q) f[q] = __fdividef(1.0f, 1.0f + __expf(-f[q]));
     }
 };
 

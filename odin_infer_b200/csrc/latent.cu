@@ -165,6 +165,8 @@ heads_linear_kernel(const TA* __restrict__ a, int a_splits, size_t a_ss, size_t 
             }
         }
     }
+    float own[HL_TOK];   // a gate per element: this thread's column of every token, loads together
+    if (gate.p != nullptr && gate.per_element && n < N) gate.columns<HL_TOK>(t0, T, h * N + n, own);
     __shared__ float factors[HL_TOK];
     if (threadIdx.x < HL_TOK) factors[threadIdx.x] = t0 + threadIdx.x < T ? gate.factor(t0 + threadIdx.x, h) : 1.0f;
     __syncthreads();
@@ -194,7 +196,7 @@ heads_linear_kernel(const TA* __restrict__ a, int a_splits, size_t a_ss, size_t 
         if (k0 + j < K) take(k0 + j, cur[j]);
 #pragma unroll
     for (int u = 0; u < HL_TOK; ++u)
-        if (t0 + u < T) out[(size_t)(t0 + u) * o_rs + (size_t)h * o_hs + n] = from_f32<TO>(acc[u] * factors[u] * gate.element(t0 + u, h, n, N));
+        if (t0 + u < T) out[(size_t)(t0 + u) * o_rs + (size_t)h * o_hs + n] = from_f32<TO>(acc[u] * (gate.per_element ? own[u] : factors[u]));
 }
 
 // Many tokens: a CTA takes 64 tokens by 64 output channels of one head, K in steps of 32 through shared memory, a thread

@@ -200,7 +200,8 @@ __device__ __forceinline__ float act_alone(int act, float z) {
     return act_gate(act, z);
 }
 
-template <bool DUAL, typename TO>
+// PER_ELEMENT: a product per head whose outputs have a gate each (the plain form)
+template <bool DUAL, typename TO, bool PER_ELEMENT = false>
 __global__ void __launch_bounds__(192)
 moe_grouped_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_w, const GroupedParams p) {
     using C = GCfg;
@@ -293,7 +294,14 @@ moe_grouped_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_const
             const float factor = (per_head && stored) ? p.gate.factor((int)i, e) : 1.0f;
 #pragma unroll 1
             for (int c0 = 0; c0 < TILE_N; c0 += 32) {
+                if (tile_n * TILE_N + c0 >= p.N) break;   // columns that do not exist
                 uint32_t r[32];
+                float g[PER_ELEMENT ? 32 : 1];
+                // whole columns of 32: their gates' loads go out together
+                const bool vec_gate = PER_ELEMENT && p.gate.aligned4 && (p.N & 3) == 0 && tile_n * TILE_N + c0 + 32 <= p.N;
+                if constexpr (PER_ELEMENT) {
+                    if (vec_gate && stored) p.gate.sigmoid32((int)i, e * p.N + tile_n * TILE_N + c0, g);
+                }
                 const uint32_t taddr = tmem_base + ((uint32_t)(quarter * 32) << 16) + c0;
                 if (DUAL) {
                     uint32_t u[32];
@@ -308,25 +316,16 @@ moe_grouped_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_const
                     if (per_head) {
 #pragma unroll
                         for (int q = 0; q < 32; ++q) r[q] = __float_as_uint(__uint_as_float(r[q]) * factor);
-                        const int j0g = tile_n * TILE_N + c0;
-                        if (p.gate.per_element && p.gate.p != nullptr && stored && j0g < p.N) {
-                            const int g0 = e * p.N + j0g;
-                            if (p.gate.aligned4 && (p.N & 3) == 0) {
+                        if (PER_ELEMENT && stored) {
+                            if (vec_gate) {
 #pragma unroll
-                                for (int q = 0; q < 32; q += 4) {
-                                    if (j0g + q < p.N) {
-                                        const float4 f = p.gate.sigmoid4_at((int)i, g0 + q);
-                                        r[q] = __float_as_uint(__uint_as_float(r[q]) * f.x);
-                                        r[q + 1] = __float_as_uint(__uint_as_float(r[q + 1]) * f.y);
-                                        r[q + 2] = __float_as_uint(__uint_as_float(r[q + 2]) * f.z);
-                                        r[q + 3] = __float_as_uint(__uint_as_float(r[q + 3]) * f.w);
-                                    }
-                                }
+                                for (int q = 0; q < 32; ++q) r[q] = __float_as_uint(__uint_as_float(r[q]) * g[q]);
                             } else {
+                                const int j0g = tile_n * TILE_N + c0;
 #pragma unroll
                                 for (int q = 0; q < 32; ++q)
                                     if (j0g + q < p.N)
-                                        r[q] = __float_as_uint(__uint_as_float(r[q]) * p.gate.sigmoid_at((int)i, g0 + q));
+                                        r[q] = __float_as_uint(__uint_as_float(r[q]) * p.gate.sigmoid_at((int)i, e * p.N + j0g + q));
                             }
                         }
                     }
@@ -431,12 +430,12 @@ int sm_count() {
     return n;
 }
 
-template <bool DUAL, typename TO>
+template <bool DUAL, typename TO, bool PER_ELEMENT = false>
 int launch_grouped(const CUtensorMap& ma, const CUtensorMap& mw, GroupedParams p, int tiles_m, cudaStream_t s, int heads = 1) {
     using C = GCfg;
     static bool configured = false;
     if (!configured) {
-        cudaError_t e = cudaFuncSetAttribute(moe_grouped_kernel<DUAL, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+        cudaError_t e = cudaFuncSetAttribute(moe_grouped_kernel<DUAL, TO, PER_ELEMENT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                              C::smem(C::MAX_STAGES));
         if (e != cudaSuccess) return (int)e;
         configured = true;
@@ -448,7 +447,7 @@ int launch_grouped(const CUtensorMap& ma, const CUtensorMap& mw, GroupedParams p
     // stages, so that enough is in flight; many CTAs: two stages, and two CTAs share an SM, one's epilogue beside the
     // other's products.  The number of CTAs follows from the shapes alone.
     p.stages = ((long long)grid.x * grid.y * grid.z <= 2LL * sm_count()) ? C::MAX_STAGES : 2;
-    odin_launch(moe_grouped_kernel<DUAL, TO>, grid, dim3(192), (size_t)C::smem(p.stages), s, ma, mw, p);
+    odin_launch(moe_grouped_kernel<DUAL, TO, PER_ELEMENT>, grid, dim3(192), (size_t)C::smem(p.stages), s, ma, mw, p);
     ODIN_LAUNCH_CHECK();
     return 0;
 }
@@ -536,8 +535,11 @@ extern "C" int odin_heads_linear_tc(const void* a, long long lda, long long a_hs
     p.error = error_flag();
     p.rows = T; p.a_hs = a_hs; p.o_hs = o_hs;
     p.gate = make_head_gate(gate, gate_dtype, gate_splits, gate_ss, gate_rs, gate_per_element);
+    const bool each = gate != nullptr && gate_per_element;
+    if (out_dtype == ODIN_F32 && each) return launch_grouped<false, float, true>(ma, mw, p, (T + BM - 1) / BM, (cudaStream_t)stream, H);
     if (out_dtype == ODIN_F32) return launch_grouped<false, float>(ma, mw, p, (T + BM - 1) / BM, (cudaStream_t)stream, H);
     if (out_dtype != ODIN_BF16) return ODIN_ERR_UNSUPPORTED;
+    if (each) return launch_grouped<false, bf16, true>(ma, mw, p, (T + BM - 1) / BM, (cudaStream_t)stream, H);
     return launch_grouped<false, bf16>(ma, mw, p, (T + BM - 1) / BM, (cudaStream_t)stream, H);
 }
 

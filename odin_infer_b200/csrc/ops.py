@@ -796,10 +796,11 @@ def gated_unit_scan(u: torch.Tensor, raw: torch.Tensor, gate_bias: torch.Tensor,
                     seq_slots: torch.Tensor, n_seqs: int, max_new: int, block_len: int = 0) -> None:
     """The same over each sequence's rows in order, the gates' products formed before: raw float32 [T, 2 n], block by block
     as gate_bias ([blocks, 2 m]) lies.  max_new: the most rows that a sequence brings; its rows are cut into blocks of
-    block_len (0: a choice by max_new) that run side by side, with the state carried from block to block."""
+    block_len (0: a choice by max_new) that run side by side, with the state carried from block to block.  raw is scratch
+    afterwards."""
     T, n = _gated_unit_args(u, gate_bias, log_decay, y, y_bias, state, out)
     assert raw.dtype == torch.float32 and raw.is_contiguous() and tuple(raw.shape) == (T, 2 * n) and max_new > 0
-    block_len = block_len or (64 if max_new <= 4096 else 256)
+    block_len = block_len or (32 if max_new <= 2048 else 64 if max_new <= 8192 else 256)
     n_blocks = (max_new + block_len - 1) // block_len
     s_own = d_own = s_first = None
     if n_blocks > 1:

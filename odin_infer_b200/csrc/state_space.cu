@@ -59,9 +59,9 @@ causal_conv_kernel(const TI* __restrict__ in, size_t in_stride, VecRef w, VecRef
 #define CONV_TOK 16
 template <typename TI, typename TO>
 __global__ void __launch_bounds__(256)
-causal_conv4_kernel(const TI* __restrict__ in, size_t in_stride, VecRef w, VecRef bias, int taps, int silu,
-                    const float* __restrict__ state, size_t state_stride, const int* __restrict__ tok_seq,
-                    const int* __restrict__ seq_start, const int* __restrict__ seq_slots, TO* __restrict__ out,
+causal_conv4_kernel(const TI* in, size_t in_stride, VecRef w, VecRef bias, int taps, int silu,
+                    const float* state, size_t state_stride, const int* __restrict__ tok_seq,
+                    const int* __restrict__ seq_start, const int* __restrict__ seq_slots, TO* out,
                     size_t out_stride, int C, int T, const float* __restrict__ in_bias) {
     pdl_trigger();
     const int t0 = blockIdx.x * CONV_TOK, t1 = min(T, t0 + CONV_TOK);
@@ -472,6 +472,47 @@ skip_gate_norm_kernel(const float* __restrict__ o, const float* __restrict__ x, 
     }
 }
 
+// out = w * o / rms(o) * sigmoid(z), one norm over the whole row of up to 4 NV blockDim.x elements (a multiple of four, everything
+// 16-byte aligned): the row and its gate stay in registers, and their loads go out together.  (o and z carry no __restrict__:
+// a load through such a const pointer counts as invariant, and the compiler may move it ahead of the wait.)
+template <typename TZ, typename TO, int NV>
+__global__ void __launch_bounds__(512)
+norm_sigmoid_kernel(const float* o, const TZ* z, size_t z_stride, VecRef w, float eps, TO* out, int n) {
+    __shared__ float shares[16];
+    pdl_trigger();
+    const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    float4 v[NV], g[NV], wv[NV];
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int j = (threadIdx.x + i * blockDim.x) * 4;
+        if (j < n) wv[i] = w.at4(j);
+    }
+    pdl_wait();
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int j = (threadIdx.x + i * blockDim.x) * 4;
+        v[i] = g[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+        if (j < n) { v[i] = ld4(o + (size_t)t * n + j); g[i] = ld4(z + (size_t)t * z_stride + j); }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) ss += (v[i].x * v[i].x + v[i].y * v[i].y) + (v[i].z * v[i].z + v[i].w * v[i].w);
+    ss = warp_sum(ss);
+    if (lane == 0) shares[warp] = ss;
+    __syncthreads();
+    ss = 0.f;
+    for (int i = 0; i < (int)(blockDim.x >> 5); ++i) ss += shares[i];
+    const float rs = 1.0f / sqrtf(ss / (float)n + eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        const int j = (threadIdx.x + i * blockDim.x) * 4;
+        if (j >= n) continue;
+        const float4 s = make_float4(1.0f + expf(-g[i].x), 1.0f + expf(-g[i].y), 1.0f + expf(-g[i].z), 1.0f + expf(-g[i].w));
+        st4(out + (size_t)t * n + j, make_float4(__fdividef(wv[i].x * (rs * v[i].x), s.x), __fdividef(wv[i].y * (rs * v[i].y), s.y),
+                                                 __fdividef(wv[i].z * (rs * v[i].z), s.z), __fdividef(wv[i].w * (rs * v[i].w), s.w)));
+    }
+}
+
 extern "C" int odin_skip_gate_norm(const float* o, const float* x, long long x_stride, const void* D, int P, const void* z,
                                    int z_dtype, long long z_stride, const void* w, int w_dtype, int groups, float eps,
                                    void* out, int out_dtype, int T, int inner, int sig_after, void* stream) {
@@ -481,6 +522,28 @@ extern "C" int odin_skip_gate_norm(const float* o, const float* x, long long x_s
     if (smem > 200 * 1024 || groups > 65535) return ODIN_ERR_UNSUPPORTED;
     cudaStream_t s = (cudaStream_t)stream;
     VecRef Dv{D, w_dtype == ODIN_BF16}, wv{w, w_dtype == ODIN_BF16};
+    if (sig_after && D == nullptr && z != nullptr && w != nullptr && groups == 1 && inner % 4 == 0 && z_stride % 4 == 0 &&
+        inner <= 4 * 4 * 512 && ((((uintptr_t)o) | ((uintptr_t)z) | ((uintptr_t)w) | ((uintptr_t)out)) & 15) == 0) {
+        // one block size per width: few rows keep a CTA busy as long as many do
+        const int nt = inner <= 512 ? 128 : inner <= 4096 ? 256 : 512;
+        const int per = (inner / 4 + nt - 1) / nt;
+#define NS(TZ, TO, NV) odin_launch(norm_sigmoid_kernel<TZ, TO, NV>, dim3(T), dim3(nt), 0, s, o, (const TZ*)z, (size_t)z_stride, wv, eps, (TO*)out, inner)
+#define NS_NV(TZ, TO)                    \
+    do {                                 \
+        if (per <= 1) NS(TZ, TO, 1);     \
+        else if (per <= 2) NS(TZ, TO, 2); \
+        else NS(TZ, TO, 4);              \
+    } while (0)
+        if (z_dtype == ODIN_BF16 && out_dtype == ODIN_BF16) NS_NV(bf16, bf16);
+        else if (z_dtype == ODIN_F32 && out_dtype == ODIN_F32) NS_NV(float, float);
+        else if (z_dtype == ODIN_F32 && out_dtype == ODIN_BF16) NS_NV(float, bf16);
+        else if (z_dtype == ODIN_BF16 && out_dtype == ODIN_F32) NS_NV(bf16, float);
+        else return ODIN_ERR_UNSUPPORTED;
+#undef NS_NV
+#undef NS
+        ODIN_LAUNCH_CHECK();
+        return 0;
+    }
     const int threads = inner / groups >= 1024 ? 256 : 128;
 #define GO(TZ, TO)                                                                                                      \
     do {                                                                                                                \
