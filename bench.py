@@ -1532,6 +1532,11 @@ def bafilorn_kernels(z: dict, T: int, peaks: dict) -> dict:
     ro, decay = torch.empty(T, RH * dv, device=dev), torch.full((RH,), 0.99, device=dev)
     for mode, name in (("fixed", "recurrence with a fixed decay (nikonex)"), ("fixed_silu", "recurrence with a fixed decay between SiLUs")):
         state.zero_()
+        if not decode:
+            note(f"{name}, {RH} heads of {dk} x {dv}, in products of tiles", timed(
+                lambda: ops.decay_blocks(q, k, v, decay, ro, state, starts, slots, n_seq, RH, dk, dv, T, silu=mode == "fixed_silu"), flush),
+                nbytes=4 * (T * 2 * RH * (dk + dv) + 2 * n_seq * RH * dk * dv), flops=T * RH * 4.0 * dk * dv)
+            state.zero_()
         note(f"{name}, {RH} heads of {dk} x {dv}" + tag, timed(
             lambda: ops.linear_recurrence(mode, q, k, None, v, decay, decay, ro, state, starts, slots, n_seq, RH, dk, dv, **blocks), flush),
             nbytes=4 * (T * 2 * RH * (dk + dv) + 2 * n_seq * RH * dk * dv), flops=T * RH * 4.0 * dk * dv)

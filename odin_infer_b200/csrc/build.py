@@ -30,6 +30,7 @@ GROUPS = {
     "rowwise": ["rowwise.cu"],
     "recurrent": ["recurrent.cu"],
     "delta_rule": ["delta_rule.cu"],
+    "decay_chunks": ["decay_chunks.cu"],
     "state_space": ["state_space.cu"],
     "gated_unit": ["gated_unit.cu"],
     "streams": ["streams.cu"],

@@ -637,6 +637,30 @@ def linear_recurrence(mode: str, q: torch.Tensor, k: torch.Tensor | None, g: tor
         "linear_recurrence", kernels=kernels)
 
 
+DECAY_BLOCK = 128   # tokens of a block of `decay_blocks`
+
+
+def decay_blocks(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, out: torch.Tensor, state: torch.Tensor,
+                 seq_start: torch.Tensor, seq_slots: torch.Tensor, n_seqs: int, n_heads: int, dk: int, dv: int, max_new: int,
+                 silu: bool = False) -> None:
+    """`linear_recurrence` with one constant decay per head ("fixed", or with silu "fixed_silu") for long prompts: every
+    sequence's rows are cut into blocks of DECAY_BLOCK tokens, whose own products (scores, outputs, what they add to the state)
+    are formed as products of tiles for all blocks at once; one small kernel carries the state from block to block.  max_new:
+    the most rows that a sequence brings.  decay: float32 [H].  The same values up to rounding (sums in another order)."""
+    for t in (q, k, v, out):
+        assert t.dtype == torch.float32 and t.stride(1) == 1
+    assert q.shape[1] == k.shape[1] == n_heads * dk and v.shape[1] == out.shape[1] == n_heads * dv and max_new > 0
+    assert state.dtype == torch.float32 and state.stride(1) == 1 and state.shape[1] >= n_heads * dk * dv
+    assert decay.dtype == torch.float32 and decay.is_contiguous() and decay.numel() == n_heads
+    n_blocks = (max_new + DECAY_BLOCK - 1) // DECAY_BLOCK
+    scratch = torch.empty(n_seqs * n_blocks, n_heads * dk * dv, dtype=torch.float32, device=q.device)
+    _check(_fn("decay_chunks", "odin_decay_blocks")(
+        _ptr(q), c_longlong(q.stride(0)), _ptr(k), c_longlong(k.stride(0)), _ptr(v), c_longlong(v.stride(0)), _ptr(decay),
+        _ptr(out), c_longlong(out.stride(0)), _ptr(state), c_longlong(state.stride(0)), _ptr(seq_start), _ptr(seq_slots),
+        c_int(n_seqs), c_int(n_heads), c_int(dk), c_int(dv), c_int(1 if silu else 0), c_int(n_blocks), _ptr(scratch), _stream()),
+        "decay_blocks", kernels=3)
+
+
 DELTA_CHUNK = 64   # tokens of a chunk of the delta rule's form for long prompts
 
 

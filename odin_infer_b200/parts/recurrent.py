@@ -27,6 +27,17 @@ def _block_len(step) -> int:
     return RECURRENCE_BLOCK if step.max_new >= BLOCKS_FROM else 0
 
 
+def _fixed_decay(step, q, k, v, decay, out, state, n_heads: int, dk: int, dv: int, silu: bool = False) -> None:
+    """The recurrence with one constant decay per head: long prompts as products of tiles over blocks of tokens, shorter steps
+    and every decode step token by token."""
+    if step.max_new >= BLOCKS_FROM:
+        ops.decay_blocks(q, k, v, decay, out, state, step.seq_start, step.seq_slots, step.n_seq_cap, n_heads, dk, dv,
+                         step.max_new, silu)
+    else:
+        ops.linear_recurrence("fixed_silu" if silu else "fixed", q, k, None, v, decay, decay, out, state, step.seq_start,
+                              step.seq_slots, step.n_seq_cap, n_heads, dk, dv)
+
+
 def _f32_view(state_bytes: torch.Tensor) -> torch.Tensor:
     """The state rows (uint8 [slots, bytes], rows any distance apart) as float32 [slots, bytes / 4]."""
     return state_bytes.view(torch.float32)
@@ -154,7 +165,7 @@ class Retention(Mixer):
         return 4 * self.H * self.D * self.V
 
     def kernel_groups(self):
-        return {"recurrent", "latent", "gemm_plain"}
+        return {"recurrent", "decay_chunks", "latent", "gemm_plain"}
 
     def forward(self, rt, step, h, entry):
         T, qk, vv = h.shape[0], self.H * self.D, self.H * self.V
@@ -167,9 +178,8 @@ class Retention(Mixer):
         ops.rope_heads(both, self.D, both, self.D, 2 * self.H, self.D, rot_dim, pairs, cos, sin, step.tok_pos,
                        scale=float(self.D) ** -0.5, scale_from_head=self.H)
         o = rt.empty(T, vv, dtype=torch.float32)
-        ops.linear_recurrence("fixed", qkvg[:, :qk], qkvg[:, qk:2 * qk], None, qkvg[:, 2 * qk:2 * qk + vv], self.decay,
-                              self.decay, o, _f32_view(step.state(entry)), step.seq_start, step.seq_slots, step.n_seq_cap,
-                              self.H, self.D, self.V, block_len=_block_len(step), max_new=step.max_new)
+        _fixed_decay(step, qkvg[:, :qk], qkvg[:, qk:2 * qk], qkvg[:, 2 * qk:2 * qk + vv], self.decay, o,
+                     _f32_view(step.state(entry)), self.H, self.D, self.V)
         y = rt.empty(T, vv)
         ops.head_unit_scale(o, None, False, qkvg[:, 2 * qk + vv:], self.eps, y, self.H, self.V)
         return rt.linear(y, self.w_o, out_dtype=torch.float32, may_split=True)
@@ -217,15 +227,14 @@ class Lightning(Mixer):
         return 4 * self.H * self.D * self.V
 
     def kernel_groups(self):
-        return {"recurrent", "state_space", "gemm_plain"}
+        return {"recurrent", "decay_chunks", "state_space", "gemm_plain"}
 
     def forward(self, rt, step, h, entry):
         T, qk, vv = h.shape[0], self.H * self.D, self.H * self.V
         qkvg = rt.linear(h, self.w_qkvg, out_dtype=torch.float32)
         o = rt.empty(T, vv, dtype=torch.float32)
-        ops.linear_recurrence("fixed_silu", qkvg[:, :qk], qkvg[:, qk:2 * qk], None, qkvg[:, 2 * qk:2 * qk + vv], self.decay,
-                              self.decay, o, _f32_view(step.state(entry)), step.seq_start, step.seq_slots, step.n_seq_cap,
-                              self.H, self.D, self.V, block_len=_block_len(step), max_new=step.max_new)
+        _fixed_decay(step, qkvg[:, :qk], qkvg[:, qk:2 * qk], qkvg[:, 2 * qk:2 * qk + vv], self.decay, o,
+                     _f32_view(step.state(entry)), self.H, self.D, self.V, silu=True)
         y = rt.empty(T, vv)
         ops.skip_gate_norm(o, None, None, self.V, qkvg[:, 2 * qk + vv:], self.norm_w, 1, self.eps, y, sigmoid_after=True)
         return rt.linear(y, self.w_o, out_dtype=torch.float32, may_split=True)

@@ -652,6 +652,47 @@ def test_fixed_decay_recurrence_between_silus(H, dk, dv, lens, blocks):
         at += n
 
 
+@pytest.mark.parametrize("silu", [False, True])
+@pytest.mark.parametrize("H,dk,dv,lens", [(3, 24, 40, (200, 1, 129)), (2, 64, 64, (256, 64)), (1, 130, 16, (300,)), (4, 128, 128, (140, 385)),
+                                          (2, 33, 70, (128, 130)), (1, 256, 200, (190,)), (5, 8, 132, (63, 64, 65, 127))])
+def test_fixed_decay_recurrence_as_products_of_tiles(H, dk, dv, lens, silu):
+    """Blocks of 128 tokens: several sequences at once from states of zeros, then a second call that goes on; a padding
+    sequence leaves its state.  Decays from one that forgets at once to one that keeps everything; an early row is loud."""
+    from odin_infer_b200.csrc import ops
+    torch.manual_seed(H + dk + dv)
+    T = sum(lens)
+    pad = 4 if dk % 4 == 0 else 3
+    x = torch.randn(T, H * (2 * dk + dv) + pad, device=DEV)
+    x[3] *= 10.0
+    decay = torch.tensor([0.0, 1.0, 0.999, 0.9, 0.5][:H] if H > 1 else [0.995])
+    slots = torch.tensor(list(range(len(lens), 0, -1)) + [0], dtype=torch.int32, device=DEV)   # the last sequence is padding
+    want, ends, at = [], [], 0
+    act = P.silu if silu else (lambda t: t)
+    for n in lens:
+        st = [torch.zeros(dk, dv, dtype=F64) for _ in range(H)]
+        qq, kk, vv = (act(t.double().cpu()) for t in x[at:at + n, :H * (2 * dk + dv)].split([H * dk, H * dk, H * dv], dim=1))
+        want.append(P.decay_walk(qq.view(n, H, dk), kk.view(n, H, dk), vv.view(n, H, dv), decay.double().tolist(), st).reshape(n, -1))
+        ends.append(torch.stack(st).reshape(-1))
+        at += n
+    want, ends = torch.cat(want), torch.stack(ends)
+    for cut in ([lambda k: (0, k)], [lambda k: (0, (2 * k + 2) // 3), lambda k: ((2 * k + 2) // 3, k)]):
+        state = torch.zeros(len(lens) + 1, H * dk * dv + 3, device=DEV)
+        state[0] = 7.0
+        for piece in cut:
+            pieces = [piece(k) for k in lens]
+            rows = torch.cat([torch.arange(sum(lens[:j]) + p0, sum(lens[:j]) + p1, device=DEV) for j, (p0, p1) in enumerate(pieces)])
+            if len(rows) == 0:
+                continue
+            sizes = [p1 - p0 for p0, p1 in pieces] + [0]
+            starts = torch.tensor([0] + np.cumsum(sizes).tolist(), dtype=torch.int32, device=DEV)
+            xr, o = x[rows].contiguous(), torch.full((len(rows), H * dv), float("nan"), device=DEV)
+            ops.decay_blocks(xr[:, :H * dk], xr[:, H * dk:2 * H * dk], xr[:, 2 * H * dk:H * (2 * dk + dv)], decay.to(DEV), o, state, starts, slots,
+                             len(lens) + 1, H, dk, dv, max(sizes), silu=silu)
+            close(o, want[rows.cpu()], 4e-6)
+        close(state[slots[:-1].long(), :H * dk * dv], ends, 4e-6)
+        assert (state[0] == 7.0).all() and (state[1:, H * dk * dv:] == 0).all()
+
+
 @pytest.mark.parametrize("T", [1, 70])
 @pytest.mark.parametrize("n,pad", [(96, 0), (100, 2), (33, 1), (2048, 4), (4100, 8), (9000, 0)])
 def test_norm_over_the_whole_row_then_a_sigmoid_gate(n, pad, T):
