@@ -46,22 +46,31 @@ __device__ __forceinline__ float db_act(float x, int silu) { return silu ? __fdi
 __device__ __forceinline__ void db_stage(float* dst, int pitch, const float* src, long long stride, int rows, int n_rows, int cols,
                                          int n_cols, int silu, int vec, const float* scale) {
     const int per = cols / 4;
-    for (int e = threadIdx.x; e < rows * per; e += blockDim.x) {
-        const int r = e / per, c = (e % per) * 4;
-        float4 x = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (r < n_rows) {
+    constexpr int U = 4;   // a thread's loads of four pieces go out together
+    for (int e0 = threadIdx.x; e0 < rows * per; e0 += blockDim.x * U) {
+        float4 x[U];
+#pragma unroll
+        for (int q = 0; q < U; ++q) {
+            const int e = e0 + q * blockDim.x, r = e / per, c = (e % per) * 4;
+            x[q] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (e >= rows * per || r >= n_rows) continue;
             const float* g = src + (size_t)r * stride + c;
-            if (vec && c + 4 <= n_cols) x = ld4(g);
+            if (vec && c + 4 <= n_cols) x[q] = ld4(g);
             else {
-                if (c < n_cols) x.x = g[0];
-                if (c + 1 < n_cols) x.y = g[1];
-                if (c + 2 < n_cols) x.z = g[2];
-                if (c + 3 < n_cols) x.w = g[3];
+                if (c < n_cols) x[q].x = g[0];
+                if (c + 1 < n_cols) x[q].y = g[1];
+                if (c + 2 < n_cols) x[q].z = g[2];
+                if (c + 3 < n_cols) x[q].w = g[3];
             }
-            if (silu) x = make_float4(db_act(x.x, 1), db_act(x.y, 1), db_act(x.z, 1), db_act(x.w, 1));
-            if (scale != nullptr) { const float f = scale[r]; x.x *= f; x.y *= f; x.z *= f; x.w *= f; }
         }
-        st4(dst + r * pitch + c, x);
+#pragma unroll
+        for (int q = 0; q < U; ++q) {
+            const int e = e0 + q * blockDim.x, r = e / per, c = (e % per) * 4;
+            if (e >= rows * per) continue;
+            if (silu) x[q] = make_float4(db_act(x[q].x, 1), db_act(x[q].y, 1), db_act(x[q].z, 1), db_act(x[q].w, 1));
+            if (scale != nullptr) { const float f = scale[r]; x[q].x *= f; x[q].y *= f; x[q].z *= f; x[q].w *= f; }
+            st4(dst + r * pitch + c, x[q]);
+        }
     }
 }
 
