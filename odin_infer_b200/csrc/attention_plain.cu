@@ -18,7 +18,7 @@
 #include <math_constants.h>
 
 #define AP_WARPS 4
-#define AP_MAX_HD 512
+#define AP_MAX_HD 1024
 
 template <typename T>
 __device__ __forceinline__ float dot_row(const float* __restrict__ q, const T* __restrict__ k, int hd);
@@ -62,14 +62,15 @@ __device__ __forceinline__ float dot_row<bf16>(const float* __restrict__ q, cons
     return acc;
 }
 
-template <typename T>
+// R: elements of a head that a lane holds (key and value heads of up to 32 R elements)
+template <typename T, int R>
 __global__ void __launch_bounds__(AP_WARPS * 32)
 attention_plain_kernel(const T* __restrict__ q, size_t q_stride, T* __restrict__ out, size_t out_stride, int T_tok,
                        int Hq, int Hkv, int hd, int vd, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
                        int page_size, const int* __restrict__ tok_pos, const int* __restrict__ tok_seq,
                        const int* __restrict__ block_table, int bt_stride, int window, int chunk, float scale,
                        float softcap, const float* __restrict__ sink) {
-    __shared__ float qs[AP_WARPS][AP_MAX_HD];
+    __shared__ float qs[AP_WARPS][32 * R];
     pdl_trigger();
     pdl_wait();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -91,9 +92,9 @@ attention_plain_kernel(const T* __restrict__ q, size_t q_stride, T* __restrict__
     if (chunk > 0) t_lo = max(t_lo, (pos / chunk) * chunk);
 
     float m = -CUDART_INF_F, l = 0.f;
-    float acc[AP_MAX_HD / 32];
+    float acc[R];
 #pragma unroll
-    for (int r = 0; r < AP_MAX_HD / 32; ++r) acc[r] = 0.f;
+    for (int r = 0; r < R; ++r) acc[r] = 0.f;
     const int* bt = block_table + (size_t)seq * bt_stride;
 
     for (int t0 = t_lo; t0 <= pos; t0 += 32) {
@@ -117,7 +118,7 @@ attention_plain_kernel(const T* __restrict__ q, size_t q_stride, T* __restrict__
         l = l * corr + warp_sum(p);
         m = m_new;
 #pragma unroll
-        for (int r = 0; r < AP_MAX_HD / 32; ++r) acc[r] *= corr;
+        for (int r = 0; r < R; ++r) acc[r] *= corr;
         const int n_here = min(32, pos - t0 + 1);
         for (int j = 0; j < n_here; ++j) {
             const float pj = __shfl_sync(0xffffffffu, p, j);
@@ -125,7 +126,7 @@ attention_plain_kernel(const T* __restrict__ q, size_t q_stride, T* __restrict__
             if (rj < 0) continue;
             const T* vrow = v_cache + (size_t)rj * vd;
 #pragma unroll
-            for (int r = 0; r < AP_MAX_HD / 32; ++r) {
+            for (int r = 0; r < R; ++r) {
                 const int d = r * 32 + lane;
                 if (d < vd) acc[r] = fmaf(pj, to_f32(vrow[d]), acc[r]);
             }
@@ -138,12 +139,12 @@ attention_plain_kernel(const T* __restrict__ q, size_t q_stride, T* __restrict__
         const float corr = expf(m - m_new);
         l = l * corr + expf(sk - m_new);
 #pragma unroll
-        for (int r = 0; r < AP_MAX_HD / 32; ++r) acc[r] *= corr;
+        for (int r = 0; r < R; ++r) acc[r] *= corr;
     }
     T* orow = out + (size_t)t * out_stride + (size_t)h * vd;
     const float inv_l = (l > 0.f) ? 1.0f / l : 0.f;
 #pragma unroll
-    for (int r = 0; r < AP_MAX_HD / 32; ++r) {
+    for (int r = 0; r < R; ++r) {
         const int d = r * 32 + lane;
         if (d < vd) orow[d] = from_f32<T>(acc[r] * inv_l);
     }
@@ -163,18 +164,23 @@ extern "C" int odin_attention_plain(const void* q, long long q_row_stride, void*
     const long long items = (long long)T * Hq;
     const long long blocks = (items + AP_WARPS - 1) / AP_WARPS;
     if (blocks > 2147483647LL) return ODIN_ERR_UNSUPPORTED;
-    if (dtype == ODIN_BF16)
-        odin_launch(attention_plain_kernel<bf16>, dim3((unsigned)blocks), dim3(AP_WARPS * 32), 0, s,
-            (const bf16*)q, (size_t)q_row_stride, (bf16*)out, (size_t)out_row_stride, T, Hq, Hkv, hd, vd,
-            (const bf16*)k_cache, (const bf16*)v_cache, page_size, tok_pos, tok_seq, block_table, bt_stride, window,
-            chunk, scale, softcap, sink);
-    else if (dtype == ODIN_F32)
-        odin_launch(attention_plain_kernel<float>, dim3((unsigned)blocks), dim3(AP_WARPS * 32), 0, s,
-            (const float*)q, (size_t)q_row_stride, (float*)out, (size_t)out_row_stride, T, Hq, Hkv, hd, vd,
-            (const float*)k_cache, (const float*)v_cache, page_size, tok_pos, tok_seq, block_table, bt_stride,
-            window, chunk, scale, softcap, sink);
-    else
-        return ODIN_ERR_UNSUPPORTED;
+#define GO(TT, R)                                                                                                       \
+    odin_launch(attention_plain_kernel<TT, R>, dim3((unsigned)blocks), dim3(AP_WARPS * 32), 0, s, (const TT*)q,          \
+                (size_t)q_row_stride, (TT*)out, (size_t)out_row_stride, T, Hq, Hkv, hd, vd, (const TT*)k_cache,           \
+                (const TT*)v_cache, page_size, tok_pos, tok_seq, block_table, bt_stride, window, chunk, scale, softcap, sink)
+#define GO_R(TT)                             \
+    do {                                     \
+        if (widest <= 128) GO(TT, 4);        \
+        else if (widest <= 256) GO(TT, 8);   \
+        else if (widest <= 512) GO(TT, 16);  \
+        else GO(TT, 32);                     \
+    } while (0)
+    const int widest = hd > vd ? hd : vd;
+    if (dtype == ODIN_BF16) GO_R(bf16);
+    else if (dtype == ODIN_F32) GO_R(float);
+    else return ODIN_ERR_UNSUPPORTED;
+#undef GO_R
+#undef GO
     ODIN_LAUNCH_CHECK();
     return 0;
 }

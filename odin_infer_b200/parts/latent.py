@@ -38,9 +38,9 @@ class LatentAttention(Mixer):
                  sink: str | None = None, gate: str | None = None, gate_per_head: bool = True):
         if min(width, n_heads, head_dim, v_head_dim, kv_rank) <= 0 or q_rank < 0 or rot_dim < 0 or rot_dim % 2:
             raise ValueError("latent attention needs positive sizes and an even rot_dim")
-        if kv_rank + rot_dim > 512:
+        if kv_rank + rot_dim > 1024:
             raise ValueError(f"latent attention: a cached row of kv_rank + rot_dim = {kv_rank + rot_dim} elements is more than "
-                             "the attention kernels take (512)")
+                             "the attention kernels take (1024)")
         if rot_dim and position_encoding is None:
             raise ValueError("latent attention with a rotated part needs a position encoding")
         self.width, self.H, self.e, self.r, self.ev = width, n_heads, head_dim, rot_dim, v_head_dim

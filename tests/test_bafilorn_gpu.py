@@ -379,7 +379,7 @@ def in_steps(mixer, rt, cache, h, cuts):
 
 LATENT_GEOMETRIES = [  # heads, dim, rotated, vdim, query latent, kv latent, rows
     (3, 20, 12, 28, 44, 36, 200), (1, 36, 4, 12, 20, 29, 131), (8, 64, 64, 32, 48, 64, 330), (4, 32, 32, 64, 72, 96, 260),
-    (5, 16, 16, 24, 33, 48, 70)]
+    (5, 16, 16, 24, 33, 48, 70), (3, 32, 64, 40, 520, 512, 90), (2, 24, 8, 16, 184, 180, 75)]
 
 
 @pytest.mark.parametrize("dtype,tol", [(torch.float32, 3e-5), (torch.bfloat16, 3e-2)])
