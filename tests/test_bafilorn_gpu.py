@@ -389,7 +389,7 @@ def test_latent_attention_alone_with_a_key_far_back(dtype, tol, geom):
     key's projection, with the input channels in another order); gates differ from element to element and token to token."""
     from odin_infer_b200.parts import PartSpec, build_part
     H, D, R, V, QR, L, n = geom
-    width, scale = 80, 40.0 / D
+    width, scale = 80, 16.0 / D
     rt = runtime(dtype)
     perm = torch.randperm(width, generator=torch.Generator().manual_seed(1))
     names = {"dq": "m.dq", "dq_norm": "m.dq.norm", "uq": "m.uq", "dkv": "m.dkv", "dkv_norm": "m.dkv.norm", "uk": "m.uk", "uv": "m.uv", "o": "m.o"}
